@@ -181,7 +181,7 @@ __device__ __forceinline__ unsigned int dropout_keep8(const DropArgs& d, unsigne
   return keep;
 }
 
-// Exact-erf GELU (nn.GELU(), VyomAI/layers/ffn.py:8) without libdevice's branchy erff: with
+// Exact-erf GELU (nn.GELU(), VyomAI/layers/ffn.py:8) instead of erff: with
 // Q(x) = 1 - Phi(|x|) = 0.5 erfc(|x| / sqrt 2) from Abramowitz-Stegun 7.1.26 (|error| <= 0.75e-7, far
 // below bf16 / tf32 resolution), gelu(x) = x Phi(x) and gelu'(x) = Phi(x) + x phi(x) share one
 // exp2 and one reciprocal (two MUFU ops), ~14 FP32 instructions per element, no divergence.
