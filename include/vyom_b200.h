@@ -27,7 +27,7 @@
 extern "C" {
 #endif
 
-#define VY_ABI_VERSION 11
+#define VY_ABI_VERSION 12
 
 #if defined(__GNUC__)
 #define VY_API __attribute__((visibility("default")))
@@ -687,6 +687,30 @@ typedef struct VyPolyNorm {
 } VyPolyNorm;
 VY_API int vy_poly_norm(const VyPolyNorm* p);
 
+/* A sublayer's close in a layer that norms its result before adding it, and the next sublayer's norm, one pass over the row, all
+ * statistics in fp32: with N_i the layer norm (x - mean) / sqrt(var + eps) * w_i + b_i (var = mean squared deviation; w / b null: 1 / 0),
+ *   s = y ? x[st] + N_1(y[st]) : x[st];   x_out = s (fp32, may be x);   copy = s (own dtype);   out = N_2(s) (own dtype)
+ * each output only when its pointer is given; st = row_index ? row_index[r] : r is the source row, outputs are written at row r.
+ * width <= 16384. */
+typedef struct VySandwichNorm {
+  int64_t rows; int32_t width;
+  const int32_t* row_index;
+  const float* x; int64_t ldx;
+  const float* y; int64_t ldy;
+  const void* w1; const void* b1; const void* w2; const void* b2; int32_t w_dtype;
+  float eps;
+  float* x_out; int64_t ld_x_out;
+  void* copy; int64_t ld_copy; int32_t copy_dtype;
+  void* out; int64_t ld_out; int32_t out_dtype;
+  void* stream;
+} VySandwichNorm;
+VY_API int vy_sandwich_norm(const VySandwichNorm* p);
+
+/* Gated feed-forward activation over interleaved pre-activations (column 2j = gate_j, 2j + 1 = up_j, the layout of VY_ACT_SWIGLU):
+ * out[r, j] = act(x[r, 2j]) * x[r, 2j + 1], fp32 arithmetic. */
+VY_API int vy_glu(int64_t rows, int32_t ff, const void* x, int64_t ldx, int32_t x_dtype, int32_t act, void* out, int64_t ld_out,
+                  int32_t out_dtype, void* stream);
+
 /* out[r, c] = act(x[r, c]) with a dtype change (the activation between two tensor-core GEMMs, computed in fp32). */
 VY_API int vy_unary(int64_t rows, int32_t cols, const void* x, int64_t ldx, int32_t x_dtype, int32_t act, void* out, int64_t ld_out,
                     int32_t out_dtype, void* stream);
@@ -718,6 +742,7 @@ VY_API int vy_kv_page_write(const VyKvWrite* p);
  * keys must already be in the pools (vy_kv_page_write). One warp per query when a sequence brings a few tokens, 64 x 64
  * register tiles for prompts; the warps of a CTA split the keys of a single-token query (decode), or, when 8 or more query
  * heads share a key / value head, the heads of the token are the rows of a 16 x 64 tile. */
+enum { VY_ATTN_SOFTMAX = 0, VY_ATTN_SIGMOID = 1 };
 typedef struct VyWinAttn {
   int32_t n_seqs, max_new;
   const int32_t* cu_tokens; const int32_t* pos0;
@@ -739,6 +764,11 @@ typedef struct VyWinAttn {
   void* stream;
   int32_t chunk;
   float out_scale; /* multiplies the output (0 = 1): a mixer's weight in a sum of mixers, applied in fp32 before the output is rounded */
+  /* VY_ATTN_SOFTMAX (0): weights are the softmax over the visible keys (and the sink). VY_ATTN_SIGMOID: the weight of a visible
+   * key is sigmoid(score), not normalised over the keys (no sink). head_scale / head_bias (one number per query head, or null):
+   * score = (q . k) * scale * head_scale[h] + head_bias[h] */
+  int32_t weight_kind;
+  const float* head_scale; const float* head_bias;
 } VyWinAttn;
 VY_API int64_t vy_window_attn_workspace_floats(int32_t n_seqs, int32_t heads, int32_t kv_heads, int32_t vdim);
 VY_API int vy_window_attn(const VyWinAttn* p);
@@ -800,6 +830,37 @@ typedef struct VyDeltaRule {
 } VyDeltaRule;
 VY_API int64_t vy_delta_rule_workspace_floats(int64_t rows, int32_t heads, int32_t kv_heads, int32_t dim);
 VY_API int vy_delta_rule(const VyDeltaRule* p);
+
+/* The gated delta rule with ONE decay per head, from the raw projections to the gated read-out, state and convolution taps carried
+ * per sequence. Per channel of q [kv_heads * dim], k [kv_heads * dim] and v [heads * vdim]: a causal convolution over `taps` inputs
+ * (weights [channels, taps], the LAST column is the current token's; zeros before position 0), then silu. Then per head h (q / k
+ * head h / (heads / kv_heads)) and token t:
+ *   qh = q / sqrt(sum q^2 + unit_eps) * dim^-1/2,  kh = k / sqrt(sum k^2 + unit_eps)
+ *   g = exp(-exp(a_log[h]) * softplus(a[t, h])),  beta = sigmoid(b[t, h])
+ *   S <- g S;  u = beta * (v - S^T kh);  S <- S + kh u^T;  o = S^T qh
+ *   out[t, h * vdim + c] = o[c] / sqrt(mean(o^2) + norm_eps) * norm[c] * gate_act(gate[t, h * vdim + c])
+ * all in fp32. state is [slots, heads, dim, vdim]; conv_state is [slots, taps, 2 kv_heads * dim + heads * vdim]: the input of position p
+ * sits in ring entry p % taps. Single-token steps are one launch; longer portions are three (all tokens' convolutions, unit vectors
+ * and decays; the recurrence, four tokens at a time; norm and gate). dim <= 256, vdim <= 512, taps <= 16. q, k, v, a, b, gate are fp32. */
+typedef struct VyGatedDelta {
+  int32_t n_seqs, max_new;
+  const int32_t* cu_tokens; const int32_t* pos0; const int32_t* slot;
+  int64_t rows;
+  const float* q; int64_t ldq; const float* k; int64_t ldk; const float* v; int64_t ldv;
+  const float* a; int64_t ld_a; const float* b; int64_t ld_b;
+  const float* gate; int64_t ld_gate; int32_t gate_act; /* VY_UACT_*; gate null: no gate */
+  const void* conv_q; const void* conv_k; const void* conv_v; int32_t conv_dtype; int32_t taps;
+  float* conv_state;
+  const void* a_log; const void* norm; int32_t w_dtype; /* a_log [heads], norm [vdim] */
+  int32_t heads, kv_heads, dim, vdim;
+  float unit_eps, norm_eps;
+  float* state;
+  void* out; int64_t ld_out; int32_t out_dtype;
+  float* workspace; int64_t workspace_floats; /* vy_gated_delta_workspace_floats(...) floats (0 for single-token steps) */
+  void* stream;
+} VyGatedDelta;
+VY_API int64_t vy_gated_delta_workspace_floats(int64_t rows, int32_t max_new, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim);
+VY_API int vy_gated_delta(const VyGatedDelta* p);
 
 /* Gated linear attention, state carried per sequence: a decay per key channel and token, no correction term. Per head h and token t:
  *   g[i] = sigmoid(a[t, h * dim + i])^(1 / tau) = exp(-softplus(-a) / tau)                       (fp32)
@@ -978,7 +1039,9 @@ VY_API int vy_depth_mix(const VyDepthMix* p);
  * head turn by pos * inv_freq[i]; the rest pass. q / k / v share a dtype (fp32 for in-place rotation at full precision).
  * Options (all 0 = the form above): half_layout pairs entry i with entry i + rot_dims / 2 instead of (2i, 2i + 1); rot_scale
  * multiplies cos and sin; with unit_rms every head of q and k is divided, after the rotation, by sqrt(mean over dim of its squares
- * + eps); q_scale / k_scale multiply the heads last. Without pools (k_pool null; no block table needed, v ignored) the rotated keys
+ * + eps); with q_norm / k_norm ([dim], shared by the heads) every head of q / k is divided by sqrt(mean over dim of its squares + eps)
+ * and multiplied by the weight BEFORE the rotation; q_scale / k_scale multiply the heads last. v may be k itself (values = the keys as
+ * projected: they are copied unnormed and unrotated). Without pools (k_pool null; no block table needed, v ignored) the rotated keys
  * go to k_out [rows, kv_heads * dim] (row stride ld_k_out, the dtype of k; may be k itself): the form recurrent mixers use. */
 typedef struct VyRopeKvWrite {
   int32_t n_seqs, max_new;
@@ -992,6 +1055,7 @@ typedef struct VyRopeKvWrite {
   int32_t half_layout, unit_rms;
   float eps, rot_scale, q_scale, k_scale;
   void* k_out; int64_t ld_k_out;
+  const void* q_norm; const void* k_norm; int32_t norm_dtype;
 } VyRopeKvWrite;
 VY_API int vy_rope_kv_write(const VyRopeKvWrite* p);
 

@@ -218,6 +218,8 @@ int vy_abi_sizeof(const char* name) {
   VY_SZ(VyMoeGather);
   VY_SZ(VyMoeCombine);
   VY_SZ(VyPolyNorm);
+  VY_SZ(VyGatedDelta);
+  VY_SZ(VySandwichNorm);
   VY_SZ(VyGatedLinAttn);
 #undef VY_SZ
   return -1;

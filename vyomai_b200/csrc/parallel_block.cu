@@ -225,6 +225,7 @@ struct RopeHeadsDev {
   int half_layout, unit_rms;
   float eps, rot_scale, q_scale, k_scale;
   void* k_out; long long ld_k_out;
+  const void* q_norm; const void* k_norm; int norm_dt;   // RMS norm with a weight [dim] before the rotation; null: none
 };
 
 __global__ void __launch_bounds__(256, 4) rope_heads_kernel(RopeHeadsDev d) {
@@ -245,15 +246,49 @@ __global__ void __launch_bounds__(256, 4) rope_heads_kernel(RopeHeadsDev d) {
       const int h = is_q ? unit : unit - b.heads;
       const void* src = is_q ? b.q : b.k;
       const long long so = row * (is_q ? b.ldq : b.ldk) + static_cast<long long>(h) * b.dim;
+      const void* nw = is_q ? d.q_norm : d.k_norm;
       float pu[4], pv[4], ps[8];
-      float ss = 0.f;
 #pragma unroll
       for (int r = 0; r < 4; ++r) {
         const int pr = lane + 32 * r;
         pu[r] = pv[r] = 0.f;
         if (pr < half) {
-          const int iu = d.half_layout ? pr : 2 * pr, iv = d.half_layout ? pr + half : 2 * pr + 1;
-          const float u = ld_as_float(src, b.in_dt, so + iu), w = ld_as_float(src, b.in_dt, so + iv);
+          pu[r] = ld_as_float(src, b.in_dt, so + (d.half_layout ? pr : 2 * pr));
+          pv[r] = ld_as_float(src, b.in_dt, so + (d.half_layout ? pr + half : 2 * pr + 1));
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < 8; ++r) {
+        const int c = lane + 32 * r;
+        ps[r] = c < rest ? ld_as_float(src, b.in_dt, so + b.rot_dims + c) : 0.f;
+      }
+      if (nw) {   // norm with a weight, then the rotation
+        float sr = 0.f;
+#pragma unroll
+        for (int r = 0; r < 4; ++r) { sr = fmaf(pu[r], pu[r], sr); sr = fmaf(pv[r], pv[r], sr); }
+#pragma unroll
+        for (int r = 0; r < 8; ++r) sr = fmaf(ps[r], ps[r], sr);
+        const float inv = 1.f / sqrtf(warp_sum(sr) / static_cast<float>(b.dim) + d.eps);
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          const int pr = lane + 32 * r;
+          if (pr < half) {
+            pu[r] *= inv * ld_as_float(nw, d.norm_dt, d.half_layout ? pr : 2 * pr);
+            pv[r] *= inv * ld_as_float(nw, d.norm_dt, d.half_layout ? pr + half : 2 * pr + 1);
+          }
+        }
+#pragma unroll
+        for (int r = 0; r < 8; ++r) {
+          const int c = lane + 32 * r;
+          if (c < rest) ps[r] *= inv * ld_as_float(nw, d.norm_dt, b.rot_dims + c);
+        }
+      }
+      float ss = 0.f;
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        const int pr = lane + 32 * r;
+        if (pr < half) {
+          const float u = pu[r], w = pv[r];
           float sn, cs;
           sincosf(static_cast<float>(pos) * b.inv_freq[pr], &sn, &cs);
           sn *= d.rot_scale;
@@ -265,11 +300,7 @@ __global__ void __launch_bounds__(256, 4) rope_heads_kernel(RopeHeadsDev d) {
         }
       }
 #pragma unroll
-      for (int r = 0; r < 8; ++r) {
-        const int c = lane + 32 * r;
-        ps[r] = c < rest ? ld_as_float(src, b.in_dt, so + b.rot_dims + c) : 0.f;
-        ss = fmaf(ps[r], ps[r], ss);
-      }
+      for (int r = 0; r < 8; ++r) ss = fmaf(ps[r], ps[r], ss);
       float f = is_q ? d.q_scale : d.k_scale;
       if (d.unit_rms) f /= sqrtf(warp_sum(ss) / static_cast<float>(b.dim) + d.eps);
       void* dst;
@@ -424,8 +455,9 @@ extern "C" int vy_rope_kv_write(const VyRopeKvWrite* p) {
   d.kp = p->k_pool; d.vp = paged ? p->v_pool : nullptr; d.pool_dt = p->pool_dtype;
   const unsigned gx = static_cast<unsigned>(p->max_new < 65535 ? p->max_new : 65535);
   const bool general = !paged || p->half_layout || p->unit_rms || (p->rot_scale != 0.f && p->rot_scale != 1.f) || (p->q_scale != 0.f && p->q_scale != 1.f) ||
-                       (p->k_scale != 0.f && p->k_scale != 1.f);
+                       (p->k_scale != 0.f && p->k_scale != 1.f) || p->q_norm || p->k_norm;
   if (general) {
+    VY_CHECK_ARG((!p->q_norm && !p->k_norm) || (dtype_ok(p->norm_dtype) && !p->unit_rms), "vy_rope_kv_write: a weighted norm before the rotation excludes unit_rms after it");
     VY_CHECK_ARG(p->dim <= 256, "vy_rope_kv_write: dim %d > 256", p->dim);
     RopeHeadsDev g;
     g.b = d;
@@ -435,6 +467,7 @@ extern "C" int vy_rope_kv_write(const VyRopeKvWrite* p) {
     g.q_scale = p->q_scale == 0.f ? 1.f : p->q_scale;
     g.k_scale = p->k_scale == 0.f ? 1.f : p->k_scale;
     g.k_out = p->k_out; g.ld_k_out = p->ld_k_out;
+    g.q_norm = p->q_norm; g.k_norm = p->k_norm; g.norm_dt = p->norm_dtype;
     // single tokens: a warp per head in flight (up to 8), few CTAs; prompts: 4 warps per token, more CTAs per SM (measured: 8 warps cost
     // prompts 0.23 -> 0.34 ms over 4 launches of 8192 tokens and saved single-token steps 29 -> 21 us)
     const int units = p->heads + p->kv_heads;

@@ -6,6 +6,8 @@
 // a sequence sits in the batch.
 #include <math.h>
 
+#include <type_traits>
+
 #include "seqmix.cuh"
 
 namespace vy {
@@ -217,6 +219,7 @@ __device__ __forceinline__ float dot_row(const void* base, int dt, long long off
 }
 
 // portions of a few tokens: one warp per query, lanes over 32 keys at a time
+template <bool SIG>
 __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(WinDev d) {
   pdl_trigger();
   pdl_wait();
@@ -236,8 +239,9 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(WinDev d) {
   int nA, lowB;
   visible_keys(d, pos, nA, lowB);
   const int count = nA + (pos + 1 - lowB);
-  float m = -INFINITY, l = 0.f;
-  if (d.sink) {
+  const float sc_mul = head_scale_of(d, h), sc_add = head_bias_of(d, h);
+  float m = -INFINITY, l = SIG ? 1.f : 0.f;
+  if (!SIG && d.sink) {
     m = ld_as_float(d.sink, d.sink_dt, h);
     l = 1.f;
   }
@@ -255,15 +259,20 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(WinDev d) {
     if (valid) {
       const int kp = c < nA ? c : lowB + (c - nA);
       row = static_cast<long long>(tab[kp / d.bs]) * d.bs + kp % d.bs;
-      sc = dot_row(d.kp, d.pool_dt, row * kstride + static_cast<long long>(g) * d.dim, d.dim, qs) * d.scale;
+      sc = dot_row(d.kp, d.pool_dt, row * kstride + static_cast<long long>(g) * d.dim, d.dim, qs) * sc_mul + sc_add;
     }
-    const float m_new = fmaxf(m, warp_max(sc));
-    const float p = valid ? expf(sc - m_new) : 0.f;
-    const float corr = m == -INFINITY ? 0.f : expf(m - m_new);
-    l = l * corr + warp_sum(p);
-    m = m_new;
+    float p;
+    if constexpr (SIG) {
+      p = valid ? sigmoidf_(sc) : 0.f;
+    } else {
+      const float m_new = fmaxf(m, warp_max(sc));
+      p = valid ? expf(sc - m_new) : 0.f;
+      const float corr = m == -INFINITY ? 0.f : expf(m - m_new);
+      l = l * corr + warp_sum(p);
+      m = m_new;
 #pragma unroll
-    for (int r = 0; r < WA_VR; ++r) acc[r] *= corr;
+      for (int r = 0; r < WA_VR; ++r) acc[r] *= corr;
+    }
     const int nv = min(32, count - tt * 32);
     for (int jj = 0; jj < nv; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
@@ -295,7 +304,8 @@ constexpr int WD_KEYS = 4;
 // reads a key or value row with one 16-byte load per 128 channels instead of four 4-byte ones.
 // HG: query heads per CTA, all reading the same key / value head (grouped heads; the single head of latent rows): a key or value
 // row is loaded once and used by the HG heads, so the pages cross L2 heads / HG times instead of heads times
-template <bool VEC, int HG>
+// SIG: sigmoid weights (no running maximum, the warps' parts simply add up)
+template <bool VEC, int HG, bool SIG>
 __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(WinDev d) {
   pdl_trigger();
   pdl_wait();
@@ -314,7 +324,7 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(WinDe
 #pragma unroll
     for (int r = 0; r < WA_VR; ++r) {
       const int col = chan(r);
-      qreg[hh][r] = col < d.dim ? ld_as_float(d.q, d.q_dt, qrow * d.ldq + static_cast<long long>(h0 + hh) * d.dim + col) * d.scale : 0.f;
+      qreg[hh][r] = col < d.dim ? ld_as_float(d.q, d.q_dt, qrow * d.ldq + static_cast<long long>(h0 + hh) * d.dim + col) * head_scale_of(d, h0 + hh) : 0.f;
     }
   const int pos = d.pos0[s];
   int nA, lowB;
@@ -324,9 +334,9 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(WinDe
   float acc[HG][WA_VR];
 #pragma unroll
   for (int hh = 0; hh < HG; ++hh) {
-    m[hh] = -INFINITY;
+    m[hh] = SIG ? 0.f : -INFINITY;
     l[hh] = 0.f;
-    if (d.sink && warp == 0) {
+    if (!SIG && d.sink && warp == 0) {
       m[hh] = ld_as_float(d.sink, d.sink_dt, h0 + hh);
       l[hh] = 1.f;
     }
@@ -397,10 +407,21 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(WinDe
     }
 #pragma unroll
     for (int hh = 0; hh < HG; ++hh) {
+      const float sc_add = head_bias_of(d, h0 + hh);
+      if constexpr (SIG) {
+        float p[WD_KEYS];
+#pragma unroll
+        for (int u = 0; u < WD_KEYS; ++u) p[u] = c0 + u < count ? sigmoidf_(warp_sum(sc[hh][u]) + sc_add) : 0.f;
+#pragma unroll
+        for (int r = 0; r < WA_VR; ++r)
+#pragma unroll
+          for (int u = 0; u < WD_KEYS; ++u) acc[hh][r] = fmaf(p[u], vv[u][r], acc[hh][r]);
+        continue;
+      }
       float m_new = m[hh];
 #pragma unroll
       for (int u = 0; u < WD_KEYS; ++u) {
-        sc[hh][u] = c0 + u < count ? warp_sum(sc[hh][u]) : -INFINITY;
+        sc[hh][u] = c0 + u < count ? warp_sum(sc[hh][u]) + sc_add : -INFINITY;
         m_new = fmaxf(m_new, sc[hh][u]);
       }
       const float corr = m[hh] == -INFINITY ? 0.f : expf(m[hh] - m_new);
@@ -445,6 +466,7 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(WinDe
     wgt[w] = ms[hh * WD_WARPS + w] == -INFINITY ? 0.f : expf(ms[hh * WD_WARPS + w] - M);
     lt = fmaf(ls[hh * WD_WARPS + w], wgt[w], lt);
   }
+  if (SIG) lt = 1.f;   // every part's maximum is 0 and its weight 1
   float og = d.out_scale / lt;
   if (d.gate) og *= sigmoidf_(ld_as_float(d.gate, d.gate_dt, qrow * d.ld_gate + h));
 #pragma unroll
@@ -904,6 +926,9 @@ extern "C" int vy_window_attn(const VyWinAttn* p) {
   d.chunk = p->chunk;
   d.out_scale = p->out_scale == 0.f ? 1.f : p->out_scale;
   d.sink = p->sink; d.sink_dt = p->sink_dtype;
+  VY_CHECK_ARG(p->weight_kind == VY_ATTN_SOFTMAX || (p->weight_kind == VY_ATTN_SIGMOID && !p->sink), "vy_window_attn: weight kind %d (sigmoid weights take no sink)", p->weight_kind);
+  d.sigmoid = p->weight_kind == VY_ATTN_SIGMOID ? 1 : 0;
+  d.head_scale = p->head_scale; d.head_bias = p->head_bias;
   d.gate = p->gate; d.ld_gate = p->ld_gate; d.gate_dt = p->gate_dtype;
   d.out = p->out; d.ld_out = p->ld_out; d.out_dt = p->out_dtype;
   cudaStream_t st = static_cast<cudaStream_t>(p->stream);
@@ -925,14 +950,19 @@ extern "C" int vy_window_attn(const VyWinAttn* p) {
     const int hg = grouped ? 4 : 1;
     const size_t smem = sizeof(float) * hg * (2 * WD_WARPS + static_cast<size_t>(WD_WARPS) * p->vdim);
     const dim3 grid(1, p->heads / hg, p->n_seqs), block(WD_WARPS * 32);
-    VY_CUDA_OK(grouped ? (vec ? launch_kernel(window_attn_decode_kernel<true, 4>, grid, block, smem, st, d)
-                              : launch_kernel(window_attn_decode_kernel<false, 4>, grid, block, smem, st, d))
-                       : (vec ? launch_kernel(window_attn_decode_kernel<true, 1>, grid, block, smem, st, d)
-                              : launch_kernel(window_attn_decode_kernel<false, 1>, grid, block, smem, st, d)));
+    const auto go = [&](auto sig) {
+      constexpr bool S = decltype(sig)::value;
+      return grouped ? (vec ? launch_kernel(window_attn_decode_kernel<true, 4, S>, grid, block, smem, st, d)
+                            : launch_kernel(window_attn_decode_kernel<false, 4, S>, grid, block, smem, st, d))
+                     : (vec ? launch_kernel(window_attn_decode_kernel<true, 1, S>, grid, block, smem, st, d)
+                            : launch_kernel(window_attn_decode_kernel<false, 1, S>, grid, block, smem, st, d));
+    };
+    VY_CUDA_OK(d.sigmoid ? go(std::true_type{}) : go(std::false_type{}));
   } else {
     const size_t smem = sizeof(float) * static_cast<size_t>(WA_WARPS) * p->dim;
-    VY_CUDA_OK(launch_kernel(window_attn_kernel, dim3((p->max_new + WA_WARPS - 1) / WA_WARPS, p->heads, p->n_seqs), dim3(WA_WARPS * 32), smem,
-                             st, d));
+    const dim3 grid((p->max_new + WA_WARPS - 1) / WA_WARPS, p->heads, p->n_seqs), block(WA_WARPS * 32);
+    VY_CUDA_OK(d.sigmoid ? launch_kernel(window_attn_kernel<true>, grid, block, smem, st, d)
+                         : launch_kernel(window_attn_kernel<false>, grid, block, smem, st, d));
   }
   VY_LAUNCH_OK();
   count_launch();

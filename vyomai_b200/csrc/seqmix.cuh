@@ -118,7 +118,12 @@ struct WinDev {
   const void* sink; int sink_dt;
   const void* gate; long long ld_gate; int gate_dt;
   void* out; long long ld_out; int out_dt;
+  int sigmoid;   // the weight of a visible key is sigmoid(score), not normalised over the keys
+  const float* head_scale; const float* head_bias;   // score = (q . k) * scale * head_scale[h] + head_bias[h]; null: 1 / 0
 };
+
+__device__ __forceinline__ float head_scale_of(const WinDev& d, int h) { return d.head_scale ? d.scale * d.head_scale[h] : d.scale; }
+__device__ __forceinline__ float head_bias_of(const WinDev& d, int h) { return d.head_bias ? d.head_bias[h] : 0.f; }
 
 // One query's visible keys at position pos: [0, nA) (kept first tokens) and [lowB, pos] (the window, or the query's chunk), disjoint
 __device__ __forceinline__ void visible_keys(const WinDev& d, int pos, int& nA, int& lowB) {

@@ -239,7 +239,8 @@ constexpr int WT_T = 256;           // threads: 16 x 16, each 4 query rows (ti +
 // BN: keys per tile. 64 halves the barriers per key; 32 lets two CTAs share an SM at 128-wide heads (the kernel is bound by
 // shared-memory and FMA latency with 8 warps, so a second CTA is what fills the issue slots)
 
-template <int MV, int BN>
+// SIG: sigmoid weights, written with the scores (no row statistics, one barrier less per key tile)
+template <int MV, int BN, bool SIG>
 __global__ void __launch_bounds__(WT_T, BN == 32 ? 2 : 1) window_attn_tiled_kernel(WinDev d, int ldq_s, int ldv_s, int dim4, int vdim4, bool qvec, bool kvvec) {
   pdl_trigger();
   pdl_wait();
@@ -281,6 +282,7 @@ __global__ void __launch_bounds__(WT_T, BN == 32 ? 2 : 1) window_attn_tiled_kern
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[r][mm][e] = 0.f;
   const long long kstride = d.k_row, vstride = d.v_row;
+  const float sc_mul = head_scale_of(d, h), sc_add = head_bias_of(d, h);
   for (int c0 = 0; c0 < count; c0 += WT_N) {
     __syncthreads();
     if (t < WT_N) {
@@ -319,9 +321,12 @@ __global__ void __launch_bounds__(WT_T, BN == 32 ? 2 : 1) window_attn_tiled_kern
         const int i = ti + 16 * r, j = tj + 16 * c;
         const int p = p_lo + i, kp = kpos_s[j];
         const bool vis = i < rows && kp >= 0 && kp <= p && (d.window <= 0 || p - kp < d.window || kp < d.keep) && (d.chunk <= 0 || kp >= p / d.chunk * d.chunk);
-        Ps[i * WT_LDP + j] = vis ? sc[r][c] * d.scale : -INFINITY;
+        const float z = fmaf(sc[r][c], sc_mul, sc_add);
+        if constexpr (SIG) Ps[i * WT_LDP + j] = vis ? sigmoidf_(z) : 0.f;
+        else Ps[i * WT_LDP + j] = vis ? z : -INFINITY;
       }
     __syncthreads();
+    if constexpr (!SIG) {
 #pragma unroll
     for (int rr = 0; rr < 8; ++rr) {
       float* pr = Ps + (8 * warp + rr) * WT_LDP;
@@ -343,6 +348,7 @@ __global__ void __launch_bounds__(WT_T, BN == 32 ? 2 : 1) window_attn_tiled_kern
       for (int mm = 0; mm < MV; ++mm)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[r][mm][e] *= cr;
+    }
     }
     const int nv = min(WT_N, (count - c0 + 3) & ~3);
     for (int j4 = 0; j4 < nv; j4 += 4) {
@@ -376,7 +382,7 @@ __global__ void __launch_bounds__(WT_T, BN == 32 ? 2 : 1) window_attn_tiled_kern
     const int i = ti + 16 * r;
     if (i >= rows) continue;
     const long long qrow = base + i0 + i;
-    float og = d.out_scale / l_s[i];
+    float og = SIG ? d.out_scale : d.out_scale / l_s[i];
     if (d.gate) og *= sigmoidf_(ld_as_float(d.gate, d.gate_dt, qrow * d.ld_gate + h));
 #pragma unroll
     for (int mm = 0; mm < MV; ++mm)
@@ -436,6 +442,10 @@ __global__ void __launch_bounds__(WH_T) window_attn_heads_kernel(WinDev d, int l
     const bool sk = d.sink && split == 0 && hh < nh;
     m[e] = sk ? ld_as_float(d.sink, d.sink_dt, h0 + hh) : -INFINITY;
     l[e] = sk ? 1.f : 0.f;
+    if (d.sigmoid) {   // every split's part has weight e^0 in the merge and the denominator is split 0's 1
+      m[e] = 0.f;
+      l[e] = split == 0 ? 1.f : 0.f;
+    }
   }
   const int kj = t & 63, hq = t >> 6;   // score phase: key kj, heads 4 hq .. 4 hq + 3; output phase: channels kj + 64 cc, same heads
   float acc[4][WH_VC];
@@ -473,13 +483,22 @@ __global__ void __launch_bounds__(WH_T) window_attn_heads_kernel(WinDev d, int l
       }
       const bool vis = krow_s[kj] >= 0;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) Ss[(4 * hq + e) * LDS_ + kj] = vis ? sc[e] * d.scale : -INFINITY;
+      for (int e = 0; e < 4; ++e) {
+        const int hh = min(h0 + 4 * hq + e, d.heads - 1);   // rows past the group hold no head: never stored
+        Ss[(4 * hq + e) * LDS_ + kj] = vis ? fmaf(sc[e], head_scale_of(d, hh), head_bias_of(d, hh)) : -INFINITY;
+      }
     }
     __syncthreads();
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       float* pr = Ss + (2 * warp + e) * LDS_;
       const float a = pr[lane], b = pr[lane + 32];
+      if (d.sigmoid) {   // parts simply add up: maximum 0, sum 1 (see the epilogue)
+        pr[lane] = a == -INFINITY ? 0.f : sigmoidf_(a);
+        pr[lane + 32] = b == -INFINITY ? 0.f : sigmoidf_(b);
+        if (lane == 0) corr_s[2 * warp + e] = 1.f;
+        continue;
+      }
       const float mn = fmaxf(m[e], warp_max(fmaxf(a, b)));
       const float cr = mn == -INFINITY ? 1.f : expf(m[e] - mn);
       const float pa = a == -INFINITY ? 0.f : expf(a - mn), pb = b == -INFINITY ? 0.f : expf(b - mn);
@@ -626,7 +645,7 @@ cudaError_t launch_window_attn_heads(const WinDev& d, int n_seqs, float* ws, lon
   return launch_kernel(window_attn_heads_merge_kernel, dim3(d.heads, n_seqs), dim3(64), 0, st, d, static_cast<int>(splits), static_cast<const float*>(ws));
 }
 
-template <int MV, int BN>
+template <int MV, int BN, bool SIG>
 static cudaError_t launch_wt(const WinDev& d, int n_seqs, int max_new, cudaStream_t st) {
   constexpr int WT_N = BN, WT_LDP = BN + 4;
   const int dim4 = (d.dim + 3) & ~3, vdim4 = (d.vdim + 3) & ~3;
@@ -639,20 +658,25 @@ static cudaError_t launch_wt(const WinDev& d, int n_seqs, int max_new, cudaStrea
   const bool kvvec = d.pool_dt == VY_F32 && d.dim % 4 == 0 && d.vdim % 4 == 0 && d.k_row % 4 == 0 && d.v_row % 4 == 0 && al(d.kp) && al(d.vp);
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
-    cudaError_t e = cudaFuncSetAttribute(window_attn_tiled_kernel<MV, BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    cudaError_t e = cudaFuncSetAttribute(window_attn_tiled_kernel<MV, BN, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return e;
     allowed = smem;
   }
-  return launch_kernel(window_attn_tiled_kernel<MV, BN>, dim3((max_new + WT_M - 1) / WT_M, d.heads, n_seqs), dim3(WT_T), smem, st, d, ldq_s, ldv_s,
+  return launch_kernel(window_attn_tiled_kernel<MV, BN, SIG>, dim3((max_new + WT_M - 1) / WT_M, d.heads, n_seqs), dim3(WT_T), smem, st, d, ldq_s, ldv_s,
                        dim4, vdim4, qvec, kvvec);
 }
 
-cudaError_t launch_window_attn_tiled(const WinDev& d, int n_seqs, int max_new, cudaStream_t st) {
+template <bool SIG>
+static cudaError_t launch_wt_any(const WinDev& d, int n_seqs, int max_new, cudaStream_t st) {
   static const int bn_env = getenv("VY_WINDOW_ATTN_BN") ? atoi(getenv("VY_WINDOW_ATTN_BN")) : 0;   // development: 32 or 64
   const bool narrow = bn_env ? bn_env == 32 : (d.dim > 64 || d.vdim > 64);   // wide heads: 64-key tiles would take the SM for one CTA
-  if (d.vdim <= 64) return narrow ? launch_wt<1, 32>(d, n_seqs, max_new, st) : launch_wt<1, 64>(d, n_seqs, max_new, st);
-  if (d.vdim <= 128) return narrow ? launch_wt<2, 32>(d, n_seqs, max_new, st) : launch_wt<2, 64>(d, n_seqs, max_new, st);
-  return launch_wt<4, 64>(d, n_seqs, max_new, st);   // vdim <= 256 (checked by the caller): the accumulators leave no room for two CTAs
+  if (d.vdim <= 64) return narrow ? launch_wt<1, 32, SIG>(d, n_seqs, max_new, st) : launch_wt<1, 64, SIG>(d, n_seqs, max_new, st);
+  if (d.vdim <= 128) return narrow ? launch_wt<2, 32, SIG>(d, n_seqs, max_new, st) : launch_wt<2, 64, SIG>(d, n_seqs, max_new, st);
+  return launch_wt<4, 64, SIG>(d, n_seqs, max_new, st);   // vdim <= 256 (checked by the caller): the accumulators leave no room for two CTAs
+}
+
+cudaError_t launch_window_attn_tiled(const WinDev& d, int n_seqs, int max_new, cudaStream_t st) {
+  return d.sigmoid ? launch_wt_any<true>(d, n_seqs, max_new, st) : launch_wt_any<false>(d, n_seqs, max_new, st);
 }
 
 }  // namespace vy

@@ -1,6 +1,6 @@
 """Sequence mixers and feed-forwards of the packed-step decoder families (models/gelutar.py, models/zugunex.py, models/vazepel.py,
-models/fubinex.py), on the packed-batch kernels of csrc/seqmix.cu, csrc/latent.cu, csrc/talking_attn.cu, csrc/parallel_block.cu and
-csrc/rowwise.cu. Each mixer is built from its config block and its weights, declares what it keeps per sequence
+models/fubinex.py, models/kifetar.py), on the packed-batch kernels of csrc/seqmix.cu, csrc/gated_delta.cu, csrc/latent.cu,
+csrc/talking_attn.cu, csrc/parallel_block.cu and csrc/rowwise.cu. Each mixer is built from its config block and its weights, declares what it keeps per sequence
 (`cache_spec`: pages of keys / values, recurrent state slots) and maps the normed layer input h [rows, width] to its
 output; the constants of a mechanism (window, kept tokens, scale, sink, decay, taps, head counts) are constructor
 arguments, so another architecture can reuse a mixer with other values.
@@ -34,15 +34,22 @@ class Projection:
         self.tensor_cores = bool(tensor_cores) and weight.dtype == torch.bfloat16 and self.in_features % 8 == 0 and self.in_features >= 32 \
             and self.out_features >= 16
 
+    def fuses_swiglu(self, x: torch.Tensor, out_dtype: torch.dtype) -> bool:
+        """Does act="swiglu" (interleaved gate / up rows) run in this product's epilogue for the input x?"""
+        return self.tensor_cores and x.dtype == torch.bfloat16 and out_dtype == torch.bfloat16 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 \
+            and self.out_features % 16 == 0 and x.shape[0] > 32
+
     def __call__(self, x: torch.Tensor, *, act: Optional[str] = None, bias: Optional[torch.Tensor] = None, scale: float = 1.0,
                  addend: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.float32, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-        N = self.out_features
+        N = self.out_features // 2 if act == "swiglu" else self.out_features
         if addend is not None and scale != 1.0:   # the two kernels order the scale and the addend differently
             raise _lib.VyomError("Projection: a scale together with an addend is not defined; fold the scale into the input")
         if out is None:
             out = torch.empty((x.shape[0], _round_up(N, 8)), device=x.device, dtype=out_dtype)[:, :N]
         tc = self.tensor_cores and x.dtype == torch.bfloat16 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 \
-            and act in (None, "none", "relu2", "gelu_tanh")
+            and act in (None, "none", "relu2", "gelu_tanh", "swiglu")
+        if act == "swiglu" and not tc:
+            raise _lib.VyomError("Projection: the gated epilogue exists on the tensor-core path only (see fuses_swiglu)")
         if tc:
             ops.gemm(x, self.weight, bias=bias, act=act, addend=addend, out=out, out_scale=scale, swap_ab=x.shape[0] <= 32)
         else:
@@ -78,7 +85,10 @@ def pack_biases(spans: List[Tuple[int, int]], total: int, biases: List[Optional[
 
 def rotary_frequencies(rot: dict, dims: int, device) -> Tuple[torch.Tensor, float]:
     """(inv_freq fp32 [dims / 2], factor on cos and sin) of a rotation block {"base", "dims", "scaling"?}. Without scaling
-    f_i = base^(-2i / dims) and the factor is 1. scaling = {"factor", "original", "fast", "slow"} stretches the slow frequencies
+    f_i = base^(-2i / dims) and the factor is 1. scaling = {"factor", "original", "low", "high"} lengthens by wavelength l_i = 2 pi / f_i (the
+    Llama 3.1 rule): f_i stays where l_i < original / high, becomes f_i / factor where l_i > original / low, and between the two
+    (1 - s) f_i / factor + s f_i with s = (original / l_i - low) / (high - low); the factor on cos / sin is 1.
+    scaling = {"factor", "original", "fast", "slow"} stretches the slow frequencies
     (YaRN): with n(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(n(fast)), 0), hi = min(ceil(n(slow)), dims - 1) and
     ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency is f_i / factor where the ramp is 1, f_i where it is 0, their
     blend between, and cos / sin are multiplied by 0.1 ln(factor) + 1."""
@@ -88,7 +98,16 @@ def rotary_frequencies(rot: dict, dims: int, device) -> Tuple[torch.Tensor, floa
     f = [base ** (-2.0 * i / dims) for i in range(half)] or [0.0]
     factor_out = 1.0
     sc = rot.get("scaling")
-    if sc and half:
+    if sc and half and "low" in sc:
+        factor, orig, low, high = (float(sc[k]) for k in ("factor", "original", "low", "high"))
+        for i in range(half):
+            wave = 2.0 * math.pi / f[i]
+            if wave > orig / low:
+                f[i] /= factor
+            elif wave >= orig / high:
+                s = (orig / wave - low) / (high - low)
+                f[i] = (1.0 - s) * f[i] / factor + s * f[i]
+    elif sc and half:
         factor, orig = float(sc["factor"]), float(sc["original"])
         turns = lambda t: dims * math.log(orig / (2.0 * math.pi * t)) / (2.0 * math.log(base))  # noqa: E731
         lo = max(math.floor(turns(float(sc["fast"]))), 0)
@@ -341,6 +360,89 @@ class RotaryAttention(Mixer):
         return self.o(a, addend=x_residual, out=x_residual)
 
 
+class SigmoidAttention(Mixer):
+    """Grouped-query attention without a softmax: the weight of a visible key is sigmoid(q . k * scale * temp_h + pb_h), not normalised
+    over the keys. q and k are projected with biases; the values are the keys as projected (no value weights); then every head of q and
+    k is RMS-normed with a weight [dim] shared by the heads and its leading rot.dims entries turn by position (entry i with entry
+    i + rot.dims / 2). mask = {"size": n}: a query sees the last n positions, its own included; no mask entry = plain causal. Each head's
+    output times sigmoid(W_g h)_h. Normed, rotated keys and raw keys (the values) live in two page pools."""
+
+    def __init__(self, cfg: dict, w: Dict[str, torch.Tensor], eps: float, act_dtype: torch.dtype, tensor_cores: bool,
+                 kv_dtype: torch.dtype = torch.float32):
+        self.heads, self.kv_heads, self.dim = int(cfg["heads"]), int(cfg["kv_heads"]), int(cfg["dim"])
+        if self.heads % self.kv_heads:
+            raise ValueError("attention: heads must be a multiple of kv_heads")
+        if int(cfg.get("vdim", self.dim)) != self.dim:
+            raise ValueError("attention: the values are the keys, so vdim equals dim")
+        rot = cfg.get("rot") or {}
+        self.rot_dims = int(rot.get("dims", 0))
+        if self.rot_dims > self.dim or self.rot_dims % 2:
+            raise ValueError("attention: rot.dims must be even and at most dim")
+        self.window = int((cfg.get("mask") or {}).get("size", 0))
+        self.scale = float(cfg["scale"])
+        self.eps, self.act_dtype, self.kv_dtype = eps, act_dtype, kv_dtype
+        self.inv_freq, self.rot_scale = rotary_frequencies(rot, self.rot_dims, w["q"].device)
+        self._in = [w["q"], w["k"], w["g"]]
+        self._in_b = [w.get("q.b"), w.get("k.b"), None]
+        self.q_norm, self.k_norm = w["q.norm"].contiguous(), w["k.norm"].contiguous()
+        self.temp = w["temp"].to(torch.float32).contiguous()
+        self.pb = w["pb"].to(torch.float32).contiguous()
+        self.o = Projection(w["o"], tensor_cores)
+
+    def input_weights(self):
+        return self._in
+
+    def input_biases(self):
+        return self._in_b
+
+    def cache_spec(self):
+        return {"pages": (self.kv_heads, self.dim, self.dim), "states": {}, "kv_dtype": self.kv_dtype}
+
+    def forward(self, parts, batch, cache):
+        q, k, g = parts
+        ops.rope_kv_write(batch, q, k, k, self.inv_freq, cache.k_pool, cache.v_pool, heads=self.heads, kv_heads=self.kv_heads, dim=self.dim,
+                          vdim=self.dim, rot_dims=self.rot_dims, layout="half", rot_scale=self.rot_scale, eps=self.eps, q_norm=self.q_norm, k_norm=self.k_norm)
+        a = ops.window_attn(batch, q, cache.k_pool, cache.v_pool, heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.dim,
+                            scale=self.scale, window=self.window, keep_first=0, gate=g, out_dtype=self.act_dtype, weights="sigmoid",
+                            head_scale=self.temp, head_bias=self.pb)
+        return self.o(a)
+
+
+class HeadDecayDeltaMixer(Mixer):
+    """Gated delta rule with one decay per head: q / k / v pass a short causal depthwise convolution and silu, q and k become unit vectors
+    per head (q also times dim^-1/2), g = exp(-exp(A_log) softplus(W_a h + dt_bias)) shrinks the head's state, sigmoid(W_b h) is the write
+    strength; each head's read-out is RMS-normed with one weight [vdim] shared by the heads and multiplied by silu(W_g h), then projected.
+    State and the convolutions' last inputs are fp32 per sequence slot (ops.gated_delta does everything between the two projections)."""
+
+    def __init__(self, cfg: dict, w: Dict[str, torch.Tensor], eps: float, act_dtype: torch.dtype, tensor_cores: bool):
+        self.heads, self.kv_heads = int(cfg["heads"]), int(cfg["kv_heads"])
+        self.dim, self.vdim, self.taps = int(cfg["dim"]), int(cfg["vdim"]), int(cfg["conv"])
+        if self.heads % self.kv_heads:
+            raise ValueError("delta mixer: heads must be a multiple of kv_heads")
+        self.eps, self.act_dtype = eps, act_dtype
+        self._in = [w["q"], w["k"], w["v"], w["g"], w["a"], w["b"]]
+        self._in_b = [None, None, None, None, w["dt_bias"], None]   # the decay's bias rides on its projection (fp32 result)
+        self.conv_w = tuple(w[n].contiguous() for n in ("q.conv", "k.conv", "v.conv"))
+        self.a_log, self.norm = w["A_log"].contiguous(), w["norm"].contiguous()
+        self.o = Projection(w["o"], tensor_cores)
+
+    def input_weights(self):
+        return self._in
+
+    def input_biases(self):
+        return self._in_b
+
+    def cache_spec(self):
+        return {"pages": None, "states": {"S": (self.heads, self.dim, self.vdim),
+                                          "conv": (self.taps, 2 * self.kv_heads * self.dim + self.heads * self.vdim)}}
+
+    def forward(self, parts, batch, cache):
+        q, k, v, g, a, b = parts
+        o = ops.gated_delta(batch, q, k, v, a, b, g, self.conv_w, cache.states["conv"], self.a_log, self.norm, cache.states["S"], heads=self.heads,
+                            kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, taps=self.taps, norm_eps=self.eps, out_dtype=self.act_dtype)
+        return self.o(o)
+
+
 class LatentAttention(Mixer):
     """Attention whose keys and values are linear images of a cached low-rank latent: per token the cache holds the RMS-normed
     latent c [rank] and one rotated key part kr [rot_dim] shared by the heads. Head h scores (qn_h . W_uk_h c + qr_h . kr) * scale
@@ -530,6 +632,22 @@ class ReluSquaredMLP(DenseMLP):
 
     def __init__(self, w: Dict[str, torch.Tensor], act_dtype: torch.dtype, tensor_cores: bool):
         super().__init__(w, act_dtype, tensor_cores, act="relu2")
+
+
+class GatedMLP:
+    """W_down (act(W_gate h) * (W_up h)), act = silu. Gate and up rows are interleaved into one product; with bf16 rows the activation runs
+    on the fp32 accumulators in the product's epilogue, otherwise on its fp32 result, rounded once for the down projection."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], act_dtype: torch.dtype, tensor_cores: bool):
+        from .gated import interleave_gate_up
+        self.up, self.down = Projection(interleave_gate_up(w["gate"], w["up"]).contiguous(), tensor_cores), Projection(w["down"], tensor_cores)
+        self.act_dtype = act_dtype
+
+    def forward(self, h: torch.Tensor) -> torch.Tensor:
+        """Returns the fp32 result (the caller norms and adds it)."""
+        if self.up.fuses_swiglu(h, self.act_dtype):
+            return self.down(self.up(h, act="swiglu", out_dtype=self.act_dtype))
+        return self.down(ops.glu(self.up(h), "silu", self.act_dtype))
 
 
 class PolyNormMLP:

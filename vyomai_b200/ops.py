@@ -977,6 +977,41 @@ def poly_norm(x: torch.Tensor, coef, *, eps: float, out_dtype: Optional[torch.dt
     return out
 
 
+def sandwich_norm(x: torch.Tensor, y: Optional[torch.Tensor] = None, norm1=None, norm2=None, *, eps: float, x_out: Optional[torch.Tensor] = None,
+                  copy_out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, row_index: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """One pass over packed fp32 rows: s = x + LayerNorm1(y) (y None: s = x), written to x_out (fp32, may be x) and copy_out (its own
+    dtype) when given; returns LayerNorm2(s) in out_dtype (norm2 None: nothing). norm1 / norm2: (weight, bias) pairs, all one dtype."""
+    w1, b1 = norm1 if norm1 is not None else (None, None)
+    w2, b2 = norm2 if norm2 is not None else (None, None)
+    ws = [t for t in (w1, b1, w2, b2) if t is not None]
+    _need_cuda(x, y, x_out, copy_out, row_index, *ws)
+    for t, n in ((x, "x"), (y, "y"), (x_out, "x_out"), (copy_out, "copy_out")):
+        if t is not None:
+            _rows2d(t, f"sandwich_norm {n}")
+    if x.dtype != torch.float32 or (y is not None and (y.dtype != torch.float32 or y.shape != x.shape)) or (x_out is not None and x_out.dtype != torch.float32):
+        raise _lib.VyomError("sandwich_norm: x, y and x_out are fp32 rows of one shape")
+    if any(t.numel() != x.shape[1] or not t.is_contiguous() or t.dtype != ws[0].dtype for t in ws):
+        raise _lib.VyomError("sandwich_norm: weights and biases are contiguous [width] and share a dtype")
+    rows = x.shape[0] if row_index is None else row_index.numel()
+    out = torch.empty((rows, x.shape[1]), device=x.device, dtype=out_dtype or torch.float32) if norm2 is not None else None
+    opt = lambda t, pre: {pre: t.data_ptr(), f"ld_{pre}": t.stride(0)} if t is not None else {}  # noqa: E731
+    _lib.call("vy_sandwich_norm", "VySandwichNorm", rows=rows, width=x.shape[1], row_index=_ptr(row_index), x=x.data_ptr(), ldx=x.stride(0), y=_ptr(y),
+              ldy=y.stride(0) if y is not None else 0, w1=_ptr(w1), b1=_ptr(b1), w2=_ptr(w2), b2=_ptr(b2), w_dtype=_dt(ws[0]) if ws else 0, eps=float(eps),
+              copy_dtype=_dt(copy_out) if copy_out is not None else 0, out_dtype=_dt(out) if out is not None else 0, stream=_stream(),
+              **opt(x_out, "x_out"), **opt(copy_out, "copy"), **opt(out, "out"))
+    return out
+
+
+def glu(x: torch.Tensor, act: str, out_dtype: torch.dtype) -> torch.Tensor:
+    """act(x[:, 0::2]) * x[:, 1::2] in fp32 (interleaved gate / up columns, the layout of gemm's act="swiglu")."""
+    _need_cuda(x)
+    _rows2d(x, "glu x")
+    ff = x.shape[1] // 2
+    out = torch.empty((x.shape[0], _round_up(ff, 8)), device=x.device, dtype=out_dtype)[:, :ff]
+    _lib.call_raw("vy_glu", x.shape[0], ff, x.data_ptr(), x.stride(0), _dt(x), UACT[act], out.data_ptr(), out.stride(0), _dt(out), _stream())
+    return out
+
+
 def unary(x: torch.Tensor, act: Optional[str], out_dtype: torch.dtype, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     _need_cuda(x, out)
     _rows2d(x, "unary x")
@@ -1010,16 +1045,24 @@ def kv_page_write(batch: PackedBatch, k: torch.Tensor, v: torch.Tensor, k_pool: 
               stream=_stream(), **batch._kw(pages=True, slots=False))
 
 
+ATTN_WEIGHTS = {"softmax": C["VY_ATTN_SOFTMAX"], "sigmoid": C["VY_ATTN_SIGMOID"]}
+
+
 def window_attn(batch: PackedBatch, q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, *, heads: int, kv_heads: int, dim: int,
                 vdim: int, scale: float, window: int, keep_first: int, sink: Optional[torch.Tensor] = None,
-                gate: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, k_row: int = 0, v_row: int = 0, chunk: int = 0, out_scale: float = 1.0) -> torch.Tensor:
+                gate: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, k_row: int = 0, v_row: int = 0, chunk: int = 0, out_scale: float = 1.0,
+                weights: str = "softmax", head_scale: Optional[torch.Tensor] = None, head_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of the step's queries over the paged pools (which already hold the step's keys): causal, restricted to the last
     `window` positions plus the first `keep_first` ones (or, with `chunk`, to the query's own block of `chunk` consecutive positions
     counted from position 0), optional per-head sink in the softmax denominator, optional per-head
-    sigmoid output gate. k_row / v_row: row strides of the pools in elements when they are not kv_heads * dim | vdim (two views of
+    sigmoid output gate. weights: "softmax", or "sigmoid" (the weight of a visible key is sigmoid(score), not normalised over keys);
+    head_scale / head_bias: fp32 [heads], score = q.k * scale * head_scale[h] + head_bias[h]. k_row / v_row: row strides of the pools in elements when they are not kv_heads * dim | vdim (two views of
     one pool)."""
-    _need_cuda(q, k_pool, v_pool, sink, gate)
+    _need_cuda(q, k_pool, v_pool, sink, gate, head_scale, head_bias)
     _rows2d(q, "window_attn q")
+    for t in (head_scale, head_bias):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != heads or not t.is_contiguous()):
+            raise _lib.VyomError("window_attn: head_scale / head_bias are contiguous fp32 [heads]")
     out = torch.empty((q.shape[0], heads * vdim), device=q.device, dtype=out_dtype or q.dtype)
     ws = None
     if batch.max_new == 1 and heads // kv_heads >= 8:   # the heads-as-rows form splits keys over CTAs and merges from a scratch buffer
@@ -1030,7 +1073,7 @@ def window_attn(batch: PackedBatch, q: torch.Tensor, k_pool: torch.Tensor, v_poo
               window=int(window), keep_first=int(keep_first), sink=_ptr(sink), sink_dtype=_dt(sink) if sink is not None else 0,
               gate=_ptr(gate), ld_gate=gate.stride(0) if gate is not None else 0, gate_dtype=_dt(gate) if gate is not None else 0,
               out=out.data_ptr(), ld_out=out.stride(0), out_dtype=_dt(out), k_row=int(k_row), v_row=int(v_row), stream=_stream(), chunk=int(chunk), out_scale=float(out_scale),
-              **batch._kw(pages=True, slots=False))
+              weight_kind=ATTN_WEIGHTS[weights], head_scale=_ptr(head_scale), head_bias=_ptr(head_bias), **batch._kw(pages=True, slots=False))
     return out
 
 
@@ -1158,12 +1201,16 @@ def depth_mix(x: torch.Tensor, y1: torch.Tensor, g1: Optional[torch.Tensor], y2:
 def rope_kv_write(batch: PackedBatch, q: Optional[torch.Tensor], k: Optional[torch.Tensor], v: Optional[torch.Tensor], inv_freq: torch.Tensor,
                   k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor], *, heads: int, kv_heads: int, dim: int, vdim: int, rot_dims: int,
                   layout: str = "pairs", rot_scale: float = 1.0, unit_rms: bool = False, eps: float = 0.0, q_scale: float = 1.0, k_scale: float = 1.0,
-                  k_out: Optional[torch.Tensor] = None) -> None:
+                  k_out: Optional[torch.Tensor] = None, q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None) -> None:
     """Rotates q in place by position, rotates k into k_pool and copies v into v_pool at each token's page row (one launch).
     layout: "pairs" turns entries (2i, 2i + 1), "half" entries (i, i + rot_dims / 2); rot_scale multiplies cos and sin; unit_rms divides
-    every rotated head of q and k by sqrt(mean of its squares + eps); q_scale / k_scale multiply the heads last. Without pools the
-    rotated keys go to k_out [rows, kv_heads * dim] (may be k itself; v is not touched)."""
-    _need_cuda(q, k, v, inv_freq, k_pool, v_pool, k_out)
+    every rotated head of q and k by sqrt(mean of its squares + eps); q_norm / k_norm (weights [dim], shared by the heads) RMS-norm every
+    head of q / k BEFORE the rotation instead; q_scale / k_scale multiply the heads last. v may be k itself (the values are the keys as
+    projected). Without pools the rotated keys go to k_out [rows, kv_heads * dim] (may be k itself; v is not touched)."""
+    _need_cuda(q, k, v, inv_freq, k_pool, v_pool, k_out, q_norm, k_norm)
+    nw = q_norm if q_norm is not None else k_norm
+    if any(t is not None and (t.numel() != dim or not t.is_contiguous() or t.dtype != nw.dtype) for t in (q_norm, k_norm)):
+        raise _lib.VyomError("rope_kv_write: q_norm / k_norm are contiguous [dim] and share a dtype")
     for t, n in ((q, "q"), (k, "k"), (v, "v"), (k_out, "k_out")):
         if t is not None:
             _rows2d(t, f"rope_kv_write {n}")
@@ -1184,6 +1231,7 @@ def rope_kv_write(batch: PackedBatch, q: Optional[torch.Tensor], k: Optional[tor
               k_pool=_ptr(k_pool), v_pool=_ptr(v_pool), pool_dtype=_dt(k_pool) if paged else 0, stream=_stream(),
               half_layout=1 if layout == "half" else 0, unit_rms=1 if unit_rms else 0, eps=float(eps), rot_scale=float(rot_scale), q_scale=float(q_scale),
               k_scale=float(k_scale), k_out=_ptr(k_out), ld_k_out=k_out.stride(0) if k_out is not None else 0,
+              q_norm=_ptr(q_norm), k_norm=_ptr(k_norm), norm_dtype=_dt(nw) if nw is not None else 0,
               **batch._kw(pages=paged, slots=False))
 
 
@@ -1334,4 +1382,42 @@ def gated_linear_attn(batch: PackedBatch, q: torch.Tensor, k: torch.Tensor, v: t
               k=k.data_ptr(), ldk=k.stride(0), v=v.data_ptr(), ldv=v.stride(0), in_dtype=_dt(q), a=a.data_ptr(), ld_a=a.stride(0), a_dtype=_dt(a),
               heads=heads, dim=dim, vdim=vdim, tau=float(tau), q_scale=float(q_scale), state=state.data_ptr(), out=out.data_ptr(), ld_out=out.stride(0),
               out_dtype=_dt(out), stream=_stream(), **batch._kw())
+    return out
+
+
+def gated_delta(batch: PackedBatch, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, b: torch.Tensor, gate: Optional[torch.Tensor],
+                conv_w, conv_state: torch.Tensor, a_log: torch.Tensor, norm: torch.Tensor, state: torch.Tensor, *, heads: int, kv_heads: int, dim: int,
+                vdim: int, taps: int, norm_eps: float, unit_eps: float = 1e-6, gate_act: Optional[str] = "silu",
+                out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """The gated delta rule with one decay per head, from the raw fp32 projections q / k [rows, kv_heads * dim], v [rows, heads * vdim],
+    a (decay logits) and b (write-strength logits) [rows, heads] to the normed, gated read-out [rows, heads * vdim]: causal convolution and
+    silu of q, k, v (conv_w: three [channels, taps] weights, last column = current token; ring conv_state [slots, taps, channels of q | k | v]),
+    unit vectors, S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, RMS norm per head with the weight `norm` [vdim], gate."""
+    cq, ck, cv = conv_w
+    _need_cuda(q, k, v, a, b, gate, cq, ck, cv, conv_state, a_log, norm, state)
+    for t, n in ((q, "q"), (k, "k"), (v, "v"), (a, "a"), (b, "b"), (gate, "gate")):
+        if t is not None:
+            _rows2d(t, f"gated_delta {n}")
+            if t.dtype != torch.float32:
+                raise _lib.VyomError(f"gated_delta: {n} is fp32")
+    qk, vv = kv_heads * dim, heads * vdim
+    if any(tuple(t.shape) != s or not t.is_contiguous() or t.dtype != cq.dtype for t, s in ((cq, (qk, taps)), (ck, (qk, taps)), (cv, (vv, taps)))):
+        raise _lib.VyomError("gated_delta: the convolution weights are contiguous [channels, taps] and share a dtype")
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (heads, dim, vdim) or conv_state.dtype != torch.float32 or \
+            not conv_state.is_contiguous() or tuple(conv_state.shape[1:]) != (taps, 2 * qk + vv):
+        raise _lib.VyomError("gated_delta: state [slots, heads, dim, vdim] and conv_state [slots, taps, channels] are contiguous fp32")
+    if a_log.numel() != heads or norm.numel() != vdim or a_log.dtype != norm.dtype or not (a_log.is_contiguous() and norm.is_contiguous()):
+        raise _lib.VyomError("gated_delta: a_log [heads] and norm [vdim] are contiguous and share a dtype")
+    if q.shape[1] < qk or k.shape[1] < qk or v.shape[1] < vv or a.shape[1] < heads or b.shape[1] < heads or (gate is not None and gate.shape[1] < vv):
+        raise _lib.VyomError("gated_delta: a projection is narrower than its heads")
+    rows = q.shape[0]
+    out = torch.empty((rows, _round_up(vv, 8)), device=q.device, dtype=out_dtype or torch.float32)[:, :vv]
+    need = int(_lib.lib().vy_gated_delta_workspace_floats(rows, batch.max_new, heads, kv_heads, dim, vdim))
+    ws = torch.empty(need, device=q.device, dtype=torch.float32) if need > 0 else None
+    _lib.call("vy_gated_delta", "VyGatedDelta", rows=rows, q=q.data_ptr(), ldq=q.stride(0), k=k.data_ptr(), ldk=k.stride(0), v=v.data_ptr(), ldv=v.stride(0),
+              a=a.data_ptr(), ld_a=a.stride(0), b=b.data_ptr(), ld_b=b.stride(0), gate=_ptr(gate), ld_gate=gate.stride(0) if gate is not None else 0,
+              gate_act=UACT[gate_act], conv_q=cq.data_ptr(), conv_k=ck.data_ptr(), conv_v=cv.data_ptr(), conv_dtype=_dt(cq), taps=taps,
+              conv_state=conv_state.data_ptr(), a_log=a_log.data_ptr(), norm=norm.data_ptr(), w_dtype=_dt(norm), heads=heads, kv_heads=kv_heads, dim=dim,
+              vdim=vdim, unit_eps=float(unit_eps), norm_eps=float(norm_eps), state=state.data_ptr(), out=out.data_ptr(), ld_out=out.stride(0),
+              out_dtype=_dt(out), workspace=_ptr(ws), workspace_floats=need, stream=_stream(), **batch._kw())
     return out

@@ -47,6 +47,11 @@ def _fubinex(path, **kw):
     return FubinexForCausalLM.from_pretrained(path, **kw)
 
 
+def _kifetar(path, **kw):
+    from .models.kifetar import KifetarForCausalLM
+    return KifetarForCausalLM.from_pretrained(path, **kw)
+
+
 def _custom_lm(path, dtype=torch.bfloat16, device=None, **kw):
     """The RMSNorm / SwiGLU / RoPE decoder (models/custom_transformer.py): config.json holds its Config fields, the checkpoint
     its state_dict."""
@@ -64,4 +69,5 @@ register_model("Gelutar", _gelutar)
 register_model("Zugunex", _zugunex)
 register_model("Vazepel", _vazepel)
 register_model("Fubinex", _fubinex)
+register_model("Kifetar", _kifetar)
 register_model("ModelForCausalLM", _custom_lm)
