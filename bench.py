@@ -1532,6 +1532,128 @@ def run_fubinex(args):
                       "clocks": sampler.result(), "l2": "160 MB buffer rewritten between timed prefill iterations"}))
 
 
+# ------------------------------------------------------------------------------------------------
+# --workload kifetar: the Kifetar decoder (sigmoid-weighted windowed attention, gated delta rule with one decay per head, sandwich
+# norms, looped layers) beside the Gelutar hybrid decoder at equal width / layer runs / vocabulary
+# ------------------------------------------------------------------------------------------------
+KIFETAR_KERNELS = ("gd_prep", "gd_scan", "gd_step", "sandwich_norm", "glu_kernel") + FUBINEX_KERNELS
+
+
+def kifetar_config(width, vocab=32768, window=512):
+    """A realistic stack of 8 layer runs: delta and attention layers in turn, six of them, the middle two looped twice; 128-wide heads
+    (4 query heads per key / value head), 128 x 128 states (2 heads per query / key head), gated feed-forward of 8/3 width."""
+    H = width // 128
+    dl = {"type": "delta", "mixer": {"heads": H, "kv_heads": max(H // 2, 1), "dim": 128, "vdim": 128, "conv": 4}}
+    at = {"type": "attention", "mixer": {"heads": H, "kv_heads": max(H // 4, 1), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
+                                         "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 1024}}}}
+    mlp = {"kind": "dense", "ff": int(8 * width / 3) // 128 * 128}
+    return {"architecture": "Kifetar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "loop": {"start": 2, "stop": 4, "times": 2},
+            "layers": [{**(dl if i % 2 == 0 else at), "mlp": mlp} for i in range(6)]}
+
+
+def measure_kifetar(dev, width, batch_prefill=4, prompt=2048, batch_decode=32, decode_steps=64, steps=5, warmup=3):
+    from vyomai_b200 import GelutarConfig, GelutarForCausalLM, KifetarConfig, KifetarForCausalLM
+    hbm, _, _, src = peaks()
+    sms = torch.cuda.get_device_properties(dev).multi_processor_count
+    fp32_tflops = sms * 128 * 2 * 1.965e9 / 1e12
+    rf = dict(fp32_tflops=fp32_tflops, hbm=hbm)
+    tokens = batch_prefill * prompt
+    cfgd = kifetar_config(width)
+    cfg = KifetarConfig(cfgd)
+    model = KifetarForCausalLM(cfg, KifetarForCausalLM.random_weights(cfg, seed=0), dtype=torch.bfloat16, device=dev)
+    runs = [cfgd["layers"][i]["type"] for i, _ in model.runs]
+    out = {"width": width, "layer_runs": runs, "vocab": cfg.vocab, "peaks": src, "fp32_tflops_nominal": round(fp32_tflops, 1)}
+    z = _packed_numbers(dev, model, cfg.vocab, batch_prefill, prompt, batch_decode, decode_steps, steps, warmup, kernels=KIFETAR_KERNELS)
+    dl, at = cfgd["layers"][0]["mixer"], cfgd["layers"][1]["mixer"]
+    ff = cfgd["layers"][0]["mlp"]["ff"]
+    n_d, n_a = runs.count("delta"), runs.count("attention")
+    n_all = n_d + n_a
+    W = at["mask"]["size"]
+    pk, dk = z["prefill_kernels"], z["decode_kernels_eager"]
+    state = dl["heads"] * dl["dim"] * dl["vdim"]
+    chan = 2 * dl["kv_heads"] * dl["dim"] + dl["heads"] * dl["vdim"]
+    vis = sum(min(p + 1, W) for p in range(prompt)) / prompt
+    z["prefill_roofline"] = {
+        "window_attn_tiled": _roof(pk, ("window_attn_tiled",), flop=n_a * tokens * at["heads"] * vis * (at["dim"] + at["vdim"]) * 2, **rf),
+        # a decay multiply and three multiply-adds per state element and token, as Gelutar's delta rule is counted
+        "gd_scan (gated delta rule)": _roof(pk, ("gd_scan",), flop=n_d * tokens * state * 7, **rf),
+        # row kernels against the copy bandwidth. gd_prep: projections in, unit vectors / values / records out (fp32)
+        "gd_prep": _roof(pk, ("gd_prep",), byts=n_d * tokens * (2 * chan + 18 * dl["heads"]) * 4, **rf),
+        # a close reads residual and result, writes residual and the next norm (bf16)
+        "sandwich_norm": _roof(pk, ("sandwich_norm",), byts=2 * n_all * tokens * width * 14, **rf),
+        "rope_heads": _roof(pk, ("rope_heads",), byts=n_a * tokens * ((at["heads"] + at["kv_heads"]) * 8 + at["kv_heads"] * 8) * at["dim"], **rf),
+        "rms_norm (delta read-out, gate; fp32 in, bf16 out)": _roof(pk, ("rms_norm",), byts=n_d * tokens * dl["heads"] * dl["vdim"] * 10, **rf),
+    }
+    z["decode_roofline"] = {
+        "window_attn_decode": _roof(dk, ("window_attn_decode", "window_attn_heads", "window_attn_heads_merge"),
+                                    byts=n_a * batch_decode * W * at["kv_heads"] * (at["dim"] + at["vdim"]) * 4, **rf),
+        "gd_step (convolutions .. gated read-out)": _roof(dk, ("gd_step",), byts=n_d * batch_decode * (state * 8 + chan * (dl["conv"] + 1) * 4), **rf),
+        "sandwich_norm": _roof(dk, ("sandwich_norm",), byts=2 * n_all * batch_decode * width * 14, **rf),
+    }
+    per_run = {i: [L.inp.weight, L.mixer.o.weight] + ([L.mlp.up.weight, L.mlp.down.weight] if L.mlp else []) for i, L in enumerate(model.layers)}
+    w_bytes = 2.0 * (sum(t.numel() for i, _ in model.runs for t in per_run[i]) + sum(o for _, o in model.runs) * model.loop_in.weight.numel() + model.embed.numel())
+    step_bytes = w_bytes + n_a * batch_decode * W * at["kv_heads"] * (at["dim"] + at["vdim"]) * 4 + n_d * batch_decode * state * 8
+    if z["decode"]["us_per_step_device"]:
+        z["decode"].update(step_algorithmic_MB=round(step_bytes / 1e6, 1),
+                           hbm_frac_device=round(step_bytes / (z["decode"]["us_per_step_device"] * 1e-6) / 1e9 / hbm, 3))
+    out["kifetar"] = z
+    del model
+    torch.cuda.empty_cache()
+    # the closest existing model: fixed-decay linear attention layers and a parallel (windowed softmax + gated delta rule) layer
+    gd = hybrid_config(width)
+    gcfg = GelutarConfig(gd)
+    gmodel = GelutarForCausalLM(gcfg, GelutarForCausalLM.random_weights(gcfg, seed=0, low_rank=64), dtype=torch.bfloat16, device=dev)
+    gz = _packed_numbers(dev, gmodel, gcfg.vocab, batch_prefill, prompt, batch_decode, decode_steps, steps, warmup, kernels=KIFETAR_KERNELS)
+    gpar = gd["layers"][3]["mixer"]
+    gl, gr = gpar["left"], gpar["right"]
+    g_par = sum(1 for L in gd["layers"] if L["type"] == "parallel")
+    g_lin = len(gd["layers"]) - g_par
+    Wg, K = gl["mask"]["size"], gl["mask"]["keep_first"]
+    gvis = sum(min(p + 1, Wg) + (min(K, p + 1 - Wg) if p + 1 > Wg else 0) for p in range(prompt)) / prompt
+    gpk, gdk = gz["prefill_kernels"], gz["decode_kernels_eager"]
+    gstate, gchan = gr["heads"] * gr["dim"] * gr["vdim"], 2 * gr["kv_heads"] * gr["dim"] + gr["heads"] * gr["vdim"]
+    glin = gd["layers"][0]["mixer"]
+    gz["prefill_roofline"] = {
+        "window_attn_tiled": _roof(gpk, ("window_attn_tiled",), flop=g_par * tokens * gl["heads"] * gvis * (gl["dim"] + gl["vdim"]) * 2, **rf),
+        "delta_rule (+ its preparing launch)": _roof(gpk, ("delta_rule",), flop=g_par * tokens * gstate * 7, **rf),
+        "causal_conv": _roof(gpk, ("causal_conv",), byts=g_par * tokens * gchan * 8, **rf),
+        # layer norms (bf16 out), the parallel layer's q / k norms and its two output norms added into the residual, the recurrences' gated read-outs
+        "rms_norm": _roof(gpk, ("rms_norm",), byts=tokens * ((2 * len(gd["layers"]) + g_lin) * width * 6 + g_lin * glin["heads"] * glin["vdim"] * 4 +
+                                                             g_par * ((gl["heads"] + gl["kv_heads"]) * gl["dim"] * 8 + 2 * width * 12 + gr["heads"] * gr["vdim"] * 10)), **rf),
+        "kv_page_write": _roof(gpk, ("kv_page_write",), byts=g_par * tokens * gl["kv_heads"] * (gl["dim"] + gl["vdim"]) * 8, **rf),
+    }
+    gz["decode_roofline"] = {
+        "window_attn (single-token forms)": _roof(gdk, ("window_attn_heads", "window_attn_heads_merge", "window_attn_decode", "window_attn"),
+                                                  byts=g_par * batch_decode * (Wg + K) * gl["kv_heads"] * (gl["dim"] + gl["vdim"]) * 4, **rf),
+        "delta_rule (its convolutions, preparing launch and norm are launches of their own)": _roof(gdk, ("delta_rule",), byts=g_par * batch_decode * gstate * 8, **rf),
+        "rms_norm": _roof(gdk, ("rms_norm",), byts=batch_decode * (2 * len(gd["layers"]) + g_lin) * width * 6, **rf),
+    }
+    out["gelutar"] = gz
+    del gmodel
+    torch.cuda.empty_cache()
+    return out
+
+
+def run_kifetar(args):
+    from vyomai_b200 import _lib
+    if int(os.environ.get("WORLD_SIZE", "1")) > 1 or args.gpus != 1:
+        print(json.dumps({"workload": "kifetar", "error": "the Kifetar decoder measurement runs on one GPU"}))
+        return
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    L = _lib.lib()
+    sampler = ClockSampler(0)
+    sampler.start()
+    n0 = L.vy_launch_count()
+    res = [_guarded(measure_kifetar, dev, int(w), steps=max(args.steps // 2, 3), warmup=max(args.warmup, 3)) for w in args.hybrid_sizes.split(",")]
+    launches = L.vy_launch_count() - n0
+    sampler.stop_flag = True
+    sampler.join(timeout=2)
+    print(json.dumps({"workload": "kifetar", "metric": "kifetar_prefill_and_decode_tokens_per_s", "n_gpus": 1, "dtype": "bf16 (fp32 residual / scores / state)",
+                      "data": "synthetic", "sizes": res, "gpu_launches_total": int(launches), "gemm_poisoned": int(L.vy_gemm_poisoned()),
+                      "clocks": sampler.result(), "l2": "160 MB buffer rewritten between timed prefill iterations"}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1539,15 +1661,16 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--workload", default="package", choices=["package", "slots", "hybrid", "latent", "talking", "fubinex"],
+    ap.add_argument("--workload", default="package", choices=["package", "slots", "hybrid", "latent", "talking", "fubinex", "kifetar"],
                     help="package: VisionLanguageModel of the reference package (1 image token + 127 text, the headline); "
                          "slots: the notebook-II form (197 image tokens in a 248-token sequence); "
                          "hybrid: prefill / decode throughput of the Gelutar hybrid decoder beside DecoderModel at equal size (1 GPU, "
                          "its own JSON line; not the headline metric); "
                          "latent: the same for the Zugunex latent-attention / mixture-of-experts decoder beside Gelutar at equal size; "
                          "talking: the same for the Vazepel parallel-layer decoder (score-exchanging attention heads) beside Zugunex; "
-                         "fubinex: the same for the Fubinex decoder (latent / block-local / gated-linear / retention mixers) beside Gelutar")
-    ap.add_argument("--hybrid-sizes", default="1024,2048", help="--workload hybrid / latent / talking / fubinex: model widths to measure")
+                         "fubinex: the same for the Fubinex decoder (latent / block-local / gated-linear / retention mixers) beside Gelutar; "
+                         "kifetar: the same for the Kifetar decoder (sigmoid-weighted attention / per-head-decay delta rule, looped layers) beside Gelutar")
+    ap.add_argument("--hybrid-sizes", default="1024,2048", help="--workload hybrid / latent / talking / fubinex / kifetar: model widths to measure")
     ap.add_argument("--no-configs-1-2", action="store_true", help="skip the encoder (C1) / ViT (C2) measurements appended at N = 1")
     ap.add_argument("--no-config5", action="store_true", help="skip the PaliGemma-scale prefill + decode measurement appended at N = 1")
     ap.add_argument("--no-slots", action="store_true", help="skip the notebook-II measurement appended at N = 1")
@@ -1570,6 +1693,8 @@ def main():
         run_talking(args)
     elif args.workload == "fubinex":
         run_fubinex(args)
+    elif args.workload == "kifetar":
+        run_kifetar(args)
     else:
         run_ours(args)
 

@@ -115,7 +115,7 @@ VY_API int vy_abi_sizeof(const char* name);
  * (kv_cache.py:355-359) are fused into the projection. k/v rows are written at token index
  * kv_dst_pos0 + l (= start_pos for a cache, 0 for a fresh buffer); q rows at l.
  *
- * Small batches (transposed_out, N <= 32 activation rows, bf16, K-major operands, K / s a multiple of 128 for some s <= 8, at most ~9.4k output features, act NONE / GELU_*, no aux / addend2 / row remaps) do not use the tensor-memory kernel at
+ * Small batches (transposed_out, N <= 32 activation rows, bf16, K-major operands, K / s a multiple of 128 for some s <= 8, at most ~9.4k output features, act NONE / GELU_* / RELU2 / SWIGLU, no aux / addend2 / row remaps) do not use the tensor-memory kernel at
  * all: csrc/gemm_skinny.cu streams the weights once through 150-400 CTAs (16 features x K / s each, mma.sync, partial sums
  * combined through the shared memory of a thread-block cluster). VY_GEMM_SKINNY=0 in the environment disables it.
  * ------------------------------------------------------------------------------------------ */
@@ -134,7 +134,8 @@ typedef struct VyGemm {
                 * up_j; N = 2 * intermediate), out has N / 2 columns: out[r, j] = silu(z[r, 2j]) * z[r, 2j+1] with z = A B^T
                 * + bias — `down_proj(act_fn(gate_proj(x)) * up_proj(x))`'s first half as ONE GEMM
                 * (VyomAI/models/custom_transformer.py:76-89; Examples/simple_vllm.ipynb FeedForward). aux (optional)
-                * receives z ([rows, N]) for vy_swiglu_bwd. No addend / transposed_out / split-K with it. */
+                * receives z ([rows, N]) for vy_swiglu_bwd. No addend / split-K with it; transposed_out only for products that the
+                * small-batch kernel below takes. */
   int32_t transposed_out;
   const void* bias; /* [cols] or NULL */
   int32_t bias_dtype;

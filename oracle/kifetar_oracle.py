@@ -3,6 +3,9 @@ sharing no code with vyomai_b200. Every function takes a WHOLE sequence from pos
 the mechanism is a recurrence; the tests compare the CUDA path (whole prompts, portions, single-token decoding, mixed batches) against
 these.
 
+The mixers and `forward` take `rnd`, a function applied to the input of every product with a weight matrix (default: none): with a
+rounding to bf16 there, the difference from the unrounded result says how far rounding alone moves a model's logits.
+
 Notation: T tokens, H heads, G key / value heads, dk / dv per-head key and value sizes.
 """
 from __future__ import annotations
@@ -57,10 +60,10 @@ def rotate_half(x, rot: Optional[dict]):
     """x [T, n, d], row t at position t: entry i of the first rot.dims turns with entry i + rot.dims / 2."""
     if not rot or not rot.get("dims"):
         return x
-    half = rot["dims"] // 2
+    half, freqs = rot["dims"] // 2, frequencies(rot)
     y = x.clone()
     for t in range(x.shape[0]):
-        for i, f in enumerate(frequencies(rot)):
+        for i, f in enumerate(freqs):
             c, s = math.cos(t * f), math.sin(t * f)
             u, v = x[t, :, i], x[t, :, i + half]
             y[t, :, i] = u * c - v * s
@@ -114,13 +117,22 @@ def gated_delta_rule(q, k, v, g, beta, state=None):
     return out
 
 
-def gated_mlp(h, gate, up, down):
-    return (silu(h @ gate.T) * (h @ up.T)) @ down.T
+def exact(x):
+    return x
+
+
+def to_bf16(x):
+    return x.to(torch.bfloat16).to(F64)
+
+
+def gated_mlp(h, gate, up, down, rnd=exact):
+    h = rnd(h)
+    return rnd(silu(h @ gate.T) * (h @ up.T)) @ down.T
 
 
 # ---- mixers and the model ----
-def attention_mixer(h, W: Dict[str, torch.Tensor], m: dict, eps: float):
-    T = h.shape[0]
+def attention_mixer(h, W: Dict[str, torch.Tensor], m: dict, eps: float, rnd=exact):
+    T, h = h.shape[0], rnd(h)
     H, G, d = m["heads"], m["kv_heads"], m["dim"]
     q = (h @ W["q"].T + W["q.b"]).view(T, H, d)
     k = (h @ W["k"].T + W["k.b"]).view(T, G, d)
@@ -129,11 +141,11 @@ def attention_mixer(h, W: Dict[str, torch.Tensor], m: dict, eps: float):
     k = rotate_half(rms(k, eps) * W["k.norm"], m.get("rot"))
     o = sigmoid_attention(q, k, v, scale=m["scale"], window=(m.get("mask") or {}).get("size", 0), temp=W["temp"], bias=W["pb"],
                           gate_logits=h @ W["g"].T)
-    return o.reshape(T, H * d) @ W["o"].T
+    return rnd(o.reshape(T, H * d)) @ W["o"].T
 
 
-def delta_mixer(h, W, m, eps):
-    T = h.shape[0]
+def delta_mixer(h, W, m, eps, rnd=exact):
+    T, h = h.shape[0], rnd(h)
     H, G, dk, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q = causal_conv(h @ W["q"].T, W["q.conv"]).view(T, G, dk)
     k = causal_conv(h @ W["k"].T, W["k.conv"]).view(T, G, dk)
@@ -143,7 +155,7 @@ def delta_mixer(h, W, m, eps):
     g = torch.exp(-torch.exp(W["A_log"]) * torch.nn.functional.softplus(h @ W["a"].T + W["dt_bias"], threshold=1e9))
     o = gated_delta_rule(q, k, v, g, beta)
     o = rms(o, eps) * W["norm"] * silu(h @ W["g"].T).view(T, H, dv)
-    return o.reshape(T, H * dv) @ W["o"].T
+    return rnd(o.reshape(T, H * dv)) @ W["o"].T
 
 
 def _sub(W, pre):
@@ -162,7 +174,7 @@ def layer_runs(cfg: dict):
     return out + [(i, False) for i in range(lp["stop"], n)]
 
 
-def forward(cfg: dict, W: Dict[str, torch.Tensor], tokens: List[int], residuals: Optional[list] = None) -> torch.Tensor:
+def forward(cfg: dict, W: Dict[str, torch.Tensor], tokens: List[int], residuals: Optional[list] = None, rnd=exact) -> torch.Tensor:
     """Logits [T, vocab] of one sequence. W: name -> float64 tensor. residuals: receives the stream after every layer run."""
     eps = cfg["norm"]["eps"]
     ln = lambda x, name: layer_norm(x, W[name], W[name + ".b"], eps)  # noqa: E731
@@ -171,15 +183,15 @@ def forward(cfg: dict, W: Dict[str, torch.Tensor], tokens: List[int], residuals:
     for i, opens in layer_runs(cfg):
         L, p = cfg["layers"][i], f"l{i}."
         if opens:
-            x = torch.cat([x, x0], 1) @ W["loop.in"].T
+            x = rnd(torch.cat([x, x0], 1)) @ W["loop.in"].T
         mixer = attention_mixer if L["type"] == "attention" else delta_mixer
-        x = x + ln(mixer(ln(x, p + "norm1"), _sub(W, p + "mix."), L["mixer"], eps), p + "norm1b")
+        x = x + ln(mixer(ln(x, p + "norm1"), _sub(W, p + "mix."), L["mixer"], eps, rnd), p + "norm1b")
         if L.get("mlp"):
-            y = gated_mlp(ln(x, p + "norm2"), W[p + "mlp.gate"], W[p + "mlp.up"], W[p + "mlp.down"])
+            y = gated_mlp(ln(x, p + "norm2"), W[p + "mlp.gate"], W[p + "mlp.up"], W[p + "mlp.down"], rnd)
             x = x + ln(y, p + "norm2b")
         if residuals is not None:
             residuals.append(x.clone())
-    return ln(x, "final.norm") @ W["embed"].T
+    return rnd(ln(x, "final.norm")) @ W["embed"].T
 
 
 def greedy(cfg, W, prompt: List[int], n_new: int):

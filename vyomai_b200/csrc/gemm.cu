@@ -298,8 +298,9 @@ extern "C" int vy_gemm(const VyGemm* p) {
     VY_CHECK_ARG(p->out != nullptr && dtype_ok(p->out_dtype), "vy_gemm: out / out_dtype invalid");
     VY_CHECK_ARG((p->act >= VY_ACT_NONE && p->act <= VY_ACT_SWIGLU) || p->act == VY_ACT_RELU2, "vy_gemm: bad act %d", p->act);
     if (p->act == VY_ACT_SWIGLU)
-      VY_CHECK_ARG((p->N & 1) == 0 && !p->addend && !p->addend2 && !p->transposed_out && p->out_row_group == 0,
-                   "vy_gemm: SWIGLU needs an even N (interleaved gate/up rows) and takes no addend / transpose / row remap");
+      VY_CHECK_ARG((p->transposed_out ? gate_act == 0 && skinny_applicable(p) : (p->N & 1) == 0) && !p->addend && !p->addend2 && p->out_row_group == 0,
+                   "vy_gemm: SWIGLU needs an even number of features (interleaved gate/up rows), takes no addend / row remap, and a transposed "
+                   "output only where the small-batch kernel serves it");
     if (p->act == VY_ACT_DGELU_ERF || p->act == VY_ACT_DGELU_TANH)
       VY_CHECK_ARG(p->aux != nullptr, "vy_gemm: DGELU epilogue needs aux (saved pre-activation)");
     if (p->bias) VY_CHECK_ARG(dtype_ok(p->bias_dtype), "vy_gemm: bad bias_dtype");

@@ -165,6 +165,15 @@ gemm_skinny_kernel(const SkinnyDev p) {
   const int f = f0 + fq;
   if (f >= p.F) return;
   const float scale = p.out_scale == 0.f ? 1.f : p.out_scale;
+  if (p.act == VY_ACT_SWIGLU) {   // features 2j, 2j + 1 are a gate and its up value: this thread holds two whole pairs (F is even)
+#pragma unroll
+    for (int j = 0; j < 4; j += 2) {
+      if (f + j >= p.F) break;
+      const float g = v[j] + (p.bias ? ld_as_float(p.bias, p.bias_dt, f + j) : 0.f), u = v[j + 1] + (p.bias ? ld_as_float(p.bias, p.bias_dt, f + j + 1) : 0.f);
+      st_from_float(p.out, p.out_dt, static_cast<long long>(tok) * p.ld_out + ((f + j) >> 1), g / (1.f + expf(-g)) * u * scale);
+    }
+    return;
+  }
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
     if (f + j < p.F) {
@@ -232,7 +241,8 @@ bool skinny_applicable(const VyGemm* p) {
   if (off) return false;
   if (p->epi != VY_EPI_LINEAR || p->in_dtype != VY_BF16 || !p->transposed_out || p->a_mn_major || p->b_mn_major) return false;
   if (p->N > 32 || p->aux || p->addend2 || p->addend_row_mod || p->out_row_group) return false;
-  if (p->act != VY_ACT_NONE && p->act != VY_ACT_GELU_ERF && p->act != VY_ACT_GELU_TANH && p->act != VY_ACT_RELU2) return false;
+  if (p->act != VY_ACT_NONE && p->act != VY_ACT_GELU_ERF && p->act != VY_ACT_GELU_TANH && p->act != VY_ACT_RELU2 && p->act != VY_ACT_SWIGLU) return false;
+  if (p->act == VY_ACT_SWIGLU && ((p->M & 1) || p->addend)) return false;
   // one wave of small CTAs is the whole point; a vocabulary-sized F (3142 feature blocks) would run ~4 latency-bound waves of
   // them and measured 2x slower than the 128-row tensor-memory tiles, which stream 77 MB at 3.5 TB/s
   if ((p->M + 15) / 16 > 4 * num_sms()) return false;

@@ -36,8 +36,10 @@ class Projection:
 
     def fuses_swiglu(self, x: torch.Tensor, out_dtype: torch.dtype) -> bool:
         """Does act="swiglu" (interleaved gate / up rows) run in this product's epilogue for the input x?"""
-        return self.tensor_cores and x.dtype == torch.bfloat16 and out_dtype == torch.bfloat16 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 \
-            and self.out_features % 16 == 0 and x.shape[0] > 32
+        if not (self.tensor_cores and x.dtype == torch.bfloat16 and out_dtype == torch.bfloat16 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
+                and self.out_features % 16 == 0):
+            return False
+        return x.shape[0] > 32 or ops.small_batch_swiglu(x.shape[0], self.weight)
 
     def __call__(self, x: torch.Tensor, *, act: Optional[str] = None, bias: Optional[torch.Tensor] = None, scale: float = 1.0,
                  addend: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.float32, out: Optional[torch.Tensor] = None) -> torch.Tensor:

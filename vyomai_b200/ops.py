@@ -94,6 +94,14 @@ def _small_batch(kw: dict) -> bool:
     return bool(_lib.lib().vy_gemm_is_small_batch(ctypes.byref(st)))
 
 
+def small_batch_swiglu(rows: int, weight: torch.Tensor) -> bool:
+    """Will gemm(x, weight, act="swiglu", swap_ab=True) be served for `rows` bf16 rows (the small-batch weight-streaming kernel)?"""
+    if weight.dtype != torch.bfloat16 or weight.stride(1) != 1:
+        return False
+    return _small_batch(dict(M=weight.shape[0], N=rows, K=weight.shape[1], in_dtype=_dt(weight), act=ACT["swiglu"], epi=C["VY_EPI_LINEAR"],
+                             transposed_out=1, A=weight.data_ptr(), lda=weight.stride(0), ldb=weight.shape[1]))
+
+
 def gemm(
     a: torch.Tensor,
     b: torch.Tensor,
@@ -133,8 +141,9 @@ def gemm(
         if rows is None:
             raise _lib.VyomError("gemm: pass `out` when using a row-group remap")
         out = torch.empty((M, N // 2 if act in ("swiglu", "geglu_tanh") else N), device=a.device, dtype=odt)
-    if act in ("swiglu", "geglu_tanh") and (swap_ab or N % 2 or out.shape[-1] != N // 2):
-        raise _lib.VyomError("gemm: act='swiglu' / 'geglu_tanh' takes interleaved gate/up rows (even N), writes N / 2 columns, no swap_ab")
+    if act in ("swiglu", "geglu_tanh") and ((swap_ab and act != "swiglu") or N % 2 or out.shape[-1] != N // 2):
+        raise _lib.VyomError("gemm: act='swiglu' / 'geglu_tanh' takes interleaved gate/up rows (even N), writes N / 2 columns; swap_ab with swiglu "
+                             "only where the small-batch kernel serves it (small_batch_swiglu)")
     if out.stride(-1) != 1:
         raise _lib.VyomError("gemm: out must be row-major")
     a_mn, lda = _major(a, "gemm a")
