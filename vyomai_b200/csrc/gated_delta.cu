@@ -429,6 +429,8 @@ __global__ void __launch_bounds__(GS_T, RM <= 16 ? 2 : 1) gd_step_kernel(GdDev d
   load_state(0);   // in flight while the convolutions and unit vectors are made
   const int qk_ch = d.kv_heads * d.dim;
   float* ring = d.conv_state + slot * d.taps * d.channels;
+  const int cur_ring = pos % d.taps;
+#pragma unroll 1
   for (int c = t; c < 2 * d.dim + d.vdim; c += GS_T) {
     const int which = c < d.dim ? 0 : c < 2 * d.dim ? 1 : 2;
     const int j = which == 0 ? c : which == 1 ? c - d.dim : c - 2 * d.dim;
@@ -437,13 +439,17 @@ __global__ void __launch_bounds__(GS_T, RM <= 16 ? 2 : 1) gd_step_kernel(GdDev d
     const float* x = which == 0 ? d.q + row * d.ldq : which == 1 ? d.k + row * d.ldk : d.v + row * d.ldv;
     const void* w = which == 0 ? d.cwq : which == 1 ? d.cwk : d.cwv;
     const float cur = x[ch];
-    float y = ld_as_float(w, d.cw_dt, static_cast<long long>(ch) * d.taps + d.taps - 1) * cur;
-    for (int lag = 1; lag < d.taps; ++lag)
-      if (pos - lag >= 0)
-        y = fmaf(ld_as_float(w, d.cw_dt, static_cast<long long>(ch) * d.taps + d.taps - 1 - lag),
-                 ring[static_cast<long long>((pos - lag) % d.taps) * d.channels + rc], y);
+    const int wo = ch * d.taps + d.taps - 1;
+    float y = ld_as_float(w, d.cw_dt, wo) * cur;
+    const int lags = min(d.taps - 1, pos);
+    int e = cur_ring;
+#pragma unroll 4
+    for (int lag = 1; lag <= lags; ++lag) {
+      e = e == 0 ? d.taps - 1 : e - 1;
+      y = fmaf(ld_as_float(w, d.cw_dt, wo - lag), ring[e * d.channels + rc], y);
+    }
     // the token's own ring entry is not one of those read above, so the CTAs of heads that share q / k do not race
-    if (which == 2 || h % rep == 0) ring[static_cast<long long>(pos % d.taps) * d.channels + rc] = cur;
+    if (which == 2 || h % rep == 0) ring[cur_ring * d.channels + rc] = cur;
     (which == 0 ? qs : which == 1 ? ks : vs)[j] = siluf_(y);
   }
   __syncthreads();
@@ -483,7 +489,7 @@ __global__ void __launch_bounds__(GS_T, RM <= 16 ? 2 : 1) gd_step_kernel(GdDev d
     __syncthreads();
 #pragma unroll
     for (int e = 0; e < 4; ++e) pr[e] = pq[e] = 0.f;
-#pragma unroll
+#pragma unroll 2
     for (int w = 0; w < GS_T / 32; ++w) {
       const float4 x = *reinterpret_cast<const float4*>(&part[w][0][4 * lane]), y = *reinterpret_cast<const float4*>(&part[w][1][4 * lane]);
       pr[0] += x.x; pr[1] += x.y; pr[2] += x.z; pr[3] += x.w;
