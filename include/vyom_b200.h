@@ -27,7 +27,7 @@
 extern "C" {
 #endif
 
-#define VY_ABI_VERSION 12
+#define VY_ABI_VERSION 13
 
 #if defined(__GNUC__)
 #define VY_API __attribute__((visibility("default")))
@@ -692,7 +692,10 @@ VY_API int vy_poly_norm(const VyPolyNorm* p);
  * statistics in fp32: with N_i the layer norm (x - mean) / sqrt(var + eps) * w_i + b_i (var = mean squared deviation; w / b null: 1 / 0),
  *   s = y ? x[st] + N_1(y[st]) : x[st];   x_out = s (fp32, may be x);   copy = s (own dtype);   out = N_2(s) (own dtype)
  * each output only when its pointer is given; st = row_index ? row_index[r] : r is the source row, outputs are written at row r.
- * width <= 16384. */
+ * norm_kind VY_CLOSE_RMS / VY_CLOSE_RMS_CENTRED: N_i is the RMS norm x / sqrt(mean(x^2) + eps) times w_i / (1 + w_i) instead (no biases).
+ * With u ([.., width] rows of their own dtype) the result that is normed is y[st] + u_coef[st] * u[st] (u_coef: one number per row):
+ * a sublayer's input, or any second result, enters with a weight per token. width <= 16384. */
+enum { VY_CLOSE_LAYER = 0, VY_CLOSE_RMS = 1, VY_CLOSE_RMS_CENTRED = 2 };
 typedef struct VySandwichNorm {
   int64_t rows; int32_t width;
   const int32_t* row_index;
@@ -704,6 +707,8 @@ typedef struct VySandwichNorm {
   void* copy; int64_t ld_copy; int32_t copy_dtype;
   void* out; int64_t ld_out; int32_t out_dtype;
   void* stream;
+  int32_t norm_kind;
+  const void* u; int64_t ld_u; int32_t u_dtype; const float* u_coef;
 } VySandwichNorm;
 VY_API int vy_sandwich_norm(const VySandwichNorm* p);
 
@@ -719,6 +724,26 @@ VY_API int vy_unary(int64_t rows, int32_t cols, const void* x, int64_t ldx, int3
 /* out[r, :] = scale * table[ids[r], :] (ids int32; an id outside [0, vocab) gives a zero row). */
 VY_API int vy_embed_rows(int32_t rows, int32_t width, int32_t vocab, const int32_t* ids, const void* table, int64_t ld_table,
                          int32_t table_dtype, float scale, void* out, int64_t ld_out, int32_t out_dtype, void* stream);
+
+/* Token embedding plus a hashed-pair embedding, packed batch:
+ *   out[r, :] = scale * table[ids[r], :] + pairs[b, :],   b = (prev * mul_prev + ids[r] * mul_cur) mod buckets
+ * prev is the sequence's token before row r: the row before, prev_state[slot] for the first row of a portion, and none for position 0,
+ * where b = buckets (the last row of the table [buckets + 1, width]). prev_state[slot] is advanced to the portion's last token. The
+ * multipliers may be any 64-bit integers >= 0 (they are reduced modulo buckets, which leaves b as it is). Ids outside [0, vocab) read
+ * zeros from the token table. */
+typedef struct VyPairEmbed {
+  int32_t n_seqs, max_new;
+  const int32_t* cu_tokens; const int32_t* pos0; const int32_t* slot;
+  const int32_t* ids;
+  int32_t width, vocab;
+  const void* table; int64_t ld_table; const void* pairs; int64_t ld_pairs; int32_t table_dtype;
+  float scale;
+  int64_t mul_prev, mul_cur; int32_t buckets;
+  int32_t* prev_state; /* [slots] */
+  void* out; int64_t ld_out; int32_t out_dtype;
+  void* stream;
+} VyPairEmbed;
+VY_API int vy_pair_embed(const VyPairEmbed* p);
 
 /* Writes the step's keys and values into paged pools [num_blocks, block_size, kv_heads, dim | vdim]: the row of
  * position p of sequence s is block_table[s * table_width + p / block_size] * block_size + p % block_size. */
@@ -770,6 +795,10 @@ typedef struct VyWinAttn {
    * score = (q . k) * scale * head_scale[h] + head_bias[h] */
   int32_t weight_kind;
   const float* head_scale; const float* head_bias;
+  /* applied to the score above, in this order: softcap > 0: s <- softcap * tanh(s / softcap); head_slope (one number per query head,
+   * or null): s <- s - head_slope[h] * (i - j), the distance between query and key. The sink gets neither. */
+  float softcap;
+  const float* head_slope;
 } VyWinAttn;
 VY_API int64_t vy_window_attn_workspace_floats(int32_t n_seqs, int32_t heads, int32_t kv_heads, int32_t vdim);
 VY_API int vy_window_attn(const VyWinAttn* p);
@@ -863,6 +892,38 @@ typedef struct VyGatedDelta {
 VY_API int64_t vy_gated_delta_workspace_floats(int64_t rows, int32_t max_new, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim);
 VY_API int vy_gated_delta(const VyGatedDelta* p);
 
+/* State-space recurrence with one decay per head and token (Mamba-2's state-space duality), from the raw projections to the gated,
+ * normed read-out, state and convolution inputs carried per sequence. Channels x [heads * vdim], b and c [groups * dim] pass a causal
+ * convolution over `taps` inputs (conv_w [channels of x | b | c, taps], the LAST column is the current token's; conv_b [channels] or
+ * null; zeros before position 0), then silu. Then per head h (b / c group h / (heads / groups)) and token t:
+ *   d = softplus(dt[t, h] + dt_bias[h]);   S <- exp(-exp(a_log[h]) d) S + d b x^T;   y = S^T c + skip[h] x        (S is dim x vdim)
+ *   u[t, h * vdim + j] = y[j] * gate_act(gate[t, h * vdim + j])                                                      (gate null: u = y)
+ *   out[t, :] = u[t, :] with each of `norm_groups` equal runs of columns divided by its own sqrt(mean of squares + norm_eps), times
+ *   norm[heads * vdim]
+ * all in fp32. state is [slots, heads, dim, vdim]; conv_state is [slots, taps, channels]: the input of position p sits in ring entry
+ * p % taps. Single-token steps are one launch (the last CTA of a sequence to finish norms its row: tickets [slots] int32, zero between
+ * launches); longer portions are three (convolutions; the recurrence chunk by chunk as products inside a chunk plus the carried state;
+ * the grouped norm). dim <= 256, vdim <= 1024, taps <= 16. x, b, c, dt, gate are fp32; the weights share w_dtype. */
+typedef struct VySsd {
+  int32_t n_seqs, max_new;
+  const int32_t* cu_tokens; const int32_t* pos0; const int32_t* slot;
+  int64_t rows;
+  const float* x; int64_t ldx; const float* b; int64_t ldb; const float* c; int64_t ldc; const float* dt; int64_t ld_dt;
+  const float* gate; int64_t ld_gate; int32_t gate_act;
+  const void* conv_w; const void* conv_b; int32_t taps;
+  float* conv_state;
+  const void* dt_bias; const void* a_log; const void* skip; const void* norm; int32_t w_dtype;
+  int32_t heads, groups, dim, vdim, norm_groups;
+  float norm_eps;
+  float* state;
+  int32_t* tickets;
+  void* out; int64_t ld_out; int32_t out_dtype;
+  float* workspace; int64_t workspace_floats; /* vy_ssd_workspace_floats(...) floats */
+  void* stream;
+} VySsd;
+VY_API int64_t vy_ssd_workspace_floats(int64_t rows, int32_t n_seqs, int32_t max_new, int32_t heads, int32_t groups, int32_t dim, int32_t vdim);
+VY_API int vy_ssd(const VySsd* p);
+
 /* Gated linear attention, state carried per sequence: a decay per key channel and token, no correction term. Per head h and token t:
  *   g[i] = sigmoid(a[t, h * dim + i])^(1 / tau) = exp(-softplus(-a) / tau)                       (fp32)
  *   S <- diag(g) S + k_t v_t^T;   o_t = S^T (q_t * q_scale)                                        (S is dim x vdim, fp32)
@@ -928,7 +989,10 @@ VY_API int vy_rope_split(const VyRopeSplit* p);
  * member and only members of the `keep_groups` best runs are eligible. The `top` largest eligible scores are chosen (ties: lowest
  * index). weight = score / (sum of the chosen scores + 1e-20) * scale, or score * scale when raw_weights is set. Writes idx
  * [rows, top] int32 and weight [rows, top] fp32 (largest first) and, when `dense` is given, dense[row, e] = weight or 0
- * ([rows, experts] fp32). experts <= 1024; groups must divide experts; top <= keep_groups * experts / groups. */
+ * ([rows, experts] fp32). experts <= 1024; groups must divide experts; top <= keep_groups * experts / groups.
+ * correction ([experts], or null): the choice is by score + correction[e], the weights are still made of the scores. The last
+ * `identity` of the experts have no weights (their output is the layer's input): dense then covers the other experts only
+ * ([rows, experts - identity]) and ident[row] receives the summed weight of the chosen identity experts. */
 enum { VY_ROUTE_SIGMOID = 0, VY_ROUTE_SOFTMAX = 1 };
 typedef struct VyMoeRoute {
   int64_t rows; int32_t experts, top;
@@ -938,6 +1002,8 @@ typedef struct VyMoeRoute {
   float* dense;
   void* stream;
   int32_t kind, groups, keep_groups, raw_weights; /* 0, 0, 0, 0: sigmoid scores, no groups, normalised weights */
+  const void* correction; int32_t correction_dtype;
+  int32_t identity; float* ident;
 } VyMoeRoute;
 VY_API int vy_moe_route(const VyMoeRoute* p);
 
@@ -983,6 +1049,8 @@ typedef struct VyMoeCombine {
   const void* addend; int64_t ld_addend; int32_t addend_dtype; /* optional [rows, width] added (the shared expert) */
   void* out; int64_t ld_out; int32_t out_dtype;
   void* stream;
+  /* optional [rows, top]: pairs whose expert idx is >= routed have no row in `part` and are left out of the sum */
+  const int32_t* idx; int32_t routed;
 } VyMoeCombine;
 VY_API int vy_moe_combine(const VyMoeCombine* p);
 
@@ -991,7 +1059,9 @@ VY_API int vy_moe_combine(const VyMoeCombine* p);
  *   g = min(gate, limit), u = clamp(up, -limit, limit), y = g * sigmoid(alpha * g) * (u + 1)        (fp32)
  *   out[row, e * ff + j] = y * dense[row * ld_dense + e] (dense null = 1; a zero weight writes 0 without reading h);
  *   out[row, experts * ff + j] = y of the shared block with shared_limit (weight 1).
- * limit <= 0 = no clamp. experts or shared_ff may be 0. */
+ * limit <= 0 = no clamp. experts or shared_ff may be 0. Options: interleaved: a block's columns are [gate_0, up_0, gate_1, up_1, ..];
+ * no_shift: the factor is u itself, not u + 1 (with alpha 1 and no limit: silu(gate) * up); shared_gate ([rows], stride ld_gate): the
+ * shared block's weight is its sigmoid. */
 typedef struct VyMoeGlu {
   int64_t rows; int32_t experts, ff, shared_ff;
   const void* h; int64_t ldh; int32_t h_dtype;
@@ -999,6 +1069,8 @@ typedef struct VyMoeGlu {
   float limit, shared_limit, alpha;
   void* out; int64_t ld_out; int32_t out_dtype;
   void* stream;
+  int32_t interleaved, no_shift;
+  const float* shared_gate; int64_t ld_gate;
 } VyMoeGlu;
 VY_API int vy_moe_glu(const VyMoeGlu* p);
 
@@ -1041,7 +1113,8 @@ VY_API int vy_depth_mix(const VyDepthMix* p);
  * Options (all 0 = the form above): half_layout pairs entry i with entry i + rot_dims / 2 instead of (2i, 2i + 1); rot_scale
  * multiplies cos and sin; with unit_rms every head of q and k is divided, after the rotation, by sqrt(mean over dim of its squares
  * + eps); with q_norm / k_norm ([dim], shared by the heads) every head of q / k is divided by sqrt(mean over dim of its squares + eps)
- * and multiplied by the weight BEFORE the rotation; q_scale / k_scale multiply the heads last. v may be k itself (values = the keys as
+ * and multiplied by the weight BEFORE the rotation; q_scale / k_scale multiply the heads last, and with q_temp_every > 0 the query at
+ * position p also by 1 + q_temp * ln(floor((p + 1) / q_temp_every) + 1). v may be k itself (values = the keys as
  * projected: they are copied unnormed and unrotated). Without pools (k_pool null; no block table needed, v ignored) the rotated keys
  * go to k_out [rows, kv_heads * dim] (row stride ld_k_out, the dtype of k; may be k itself): the form recurrent mixers use. */
 typedef struct VyRopeKvWrite {
@@ -1057,6 +1130,7 @@ typedef struct VyRopeKvWrite {
   float eps, rot_scale, q_scale, k_scale;
   void* k_out; int64_t ld_k_out;
   const void* q_norm; const void* k_norm; int32_t norm_dtype;
+  float q_temp; int32_t q_temp_every;
 } VyRopeKvWrite;
 VY_API int vy_rope_kv_write(const VyRopeKvWrite* p);
 

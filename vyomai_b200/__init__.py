@@ -21,4 +21,5 @@ from .models.zugunex import ZugunexConfig, ZugunexForCausalLM  # noqa: F401
 from .models.vazepel import VazepelConfig, VazepelForCausalLM  # noqa: F401
 from .models.fubinex import FubinexConfig, FubinexForCausalLM  # noqa: F401
 from .models.kifetar import KifetarConfig, KifetarForCausalLM  # noqa: F401
+from .models.zaparax import ZaparaxConfig, ZaparaxForCausalLM  # noqa: F401
 from .registry import load_model, register_model  # noqa: F401

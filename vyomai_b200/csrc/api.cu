@@ -221,6 +221,8 @@ int vy_abi_sizeof(const char* name) {
   VY_SZ(VyGatedDelta);
   VY_SZ(VySandwichNorm);
   VY_SZ(VyGatedLinAttn);
+  VY_SZ(VyPairEmbed);
+  VY_SZ(VySsd);
 #undef VY_SZ
   return -1;
 }

@@ -41,7 +41,6 @@ struct GdDev {
 
 constexpr int GD_B = 4;          // tokens per block of the recurrence
 constexpr int GD_REC = 16;       // floats per (token, head) record: [-beta G, beta, G, G_3 / G | 4 of the u chain | 4 of the o chain | G_3, pad]
-constexpr float GD_MIN_LOG = -1e4f;   // exp of it is 0 in fp32; keeps sums and differences of log decays finite
 
 // 32 values per lane -> the warp's sum of value number `lane`
 __device__ __forceinline__ float reduce_scatter32(float (&v)[32], int lane) {
@@ -58,7 +57,7 @@ __device__ __forceinline__ float reduce_scatter32(float (&v)[32], int lane) {
 }
 
 __device__ __forceinline__ float log_decay(const GdDev& d, int h, float a) {
-  return fmaxf(-expf(ld_as_float(d.a_log, d.w_dt, h)) * softplusf_(a), GD_MIN_LOG);
+  return fmaxf(-expf(ld_as_float(d.a_log, d.w_dt, h)) * softplusf_(a), MIN_LOG_DECAY);
 }
 
 // silu of the convolution of one channel at tokens i0 .. i0 + 3 of the portion (TP >= taps; positions before the portion from the ring)

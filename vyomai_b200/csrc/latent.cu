@@ -117,6 +117,8 @@ struct RouteDev {
   float scale;
   int* idx; float* weight; float* dense;
   int kind, groups, keep_groups, raw;
+  const void* corr; int corr_dt;   // added to the scores for the choice only
+  int identity; float* ident;      // the last `identity` experts have no weights: their chosen weights are summed per row
 };
 
 constexpr int ROUTE_WARPS = 4;
@@ -141,6 +143,7 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(RouteDev d)
   const long long r = static_cast<long long>(blockIdx.x) * ROUTE_WARPS + warp;
   if (r >= d.rows) return;
   float* sc = route_smem + warp * (d.experts + d.groups);
+  const int routed = d.experts - d.identity;
   float zmax = -INFINITY, zsum = 0.f;
   if (d.kind == VY_ROUTE_SOFTMAX) {
     for (int e = lane; e < d.experts; e += 32) zmax = fmaxf(zmax, d.logits[r * d.ld + e]);
@@ -151,7 +154,8 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(RouteDev d)
   for (int e = lane; e < d.experts; e += 32) {
     const float z = d.logits[r * d.ld + e];
     sc[e] = d.kind == VY_ROUTE_SOFTMAX ? expf(z - zmax) / zsum : sigmoidf_(z);
-    if (d.dense) d.dense[r * d.experts + e] = 0.f;
+    if (d.corr) sc[e] += ld_as_float(d.corr, d.corr_dt, e);
+    if (d.dense && e < routed) d.dense[r * routed + e] = 0.f;
   }
   __syncwarp();
   if (d.groups > 1) {
@@ -175,7 +179,7 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(RouteDev d)
       __syncwarp();
     }
     for (int e = lane; e < d.experts; e += 32)
-      if (gs[e / per] != -INFINITY) sc[e] = -INFINITY;   // scores are positive, so a kept group never reads -inf here by itself
+      if (gs[e / per] != -INFINITY) sc[e] = -INFINITY;   // scores (and corrections) are finite, so a kept group never reads -inf here by itself
     __syncwarp();
   }
   float sum = 0.f;
@@ -189,6 +193,11 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(RouteDev d)
       if (v > bv) { bv = v; bi = e; }   // ascending e: the lowest index of equal values stays
     }
     warp_argmax(bv, bi);
+    bi = min(bi, d.experts - 1);   // logits that are not numbers leave no maximum
+    if (d.corr) {   // the weight is the score without the correction
+      const float z = d.logits[r * d.ld + bi];
+      bv = d.kind == VY_ROUTE_SOFTMAX ? expf(z - zmax) / zsum : sigmoidf_(z);
+    }
     sum += bv;
     if (lane == (k & 31)) { my_val = bv; my_idx = bi; }
     if (lane == 0) sc[bi] = -INFINITY;
@@ -204,10 +213,17 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(RouteDev d)
   }
   __syncwarp();
   const float norm = d.raw ? d.scale : d.scale / (sum + 1e-20f);
+  float iw = 0.f;
   for (int k = lane; k < d.top; k += 32) {
     const float w = d.weight[r * d.top + k] * norm;
     d.weight[r * d.top + k] = w;
-    if (d.dense) d.dense[r * d.experts + d.idx[r * d.top + k]] = w;
+    const int e = d.idx[r * d.top + k];
+    if (e >= routed) iw += w;
+    else if (d.dense) d.dense[r * routed + e] = w;
+  }
+  if (d.ident) {
+    iw = warp_sum(iw);
+    if (lane == 0) d.ident[r] = iw;
   }
 }
 
@@ -331,6 +347,7 @@ struct CombineDev {
   const void* part; long long ld_part; int part_dt;
   const void* addend; long long ld_addend; int addend_dt;
   void* out; long long ld_out; int out_dt;
+  const int* idx; int routed;   // pairs with an expert >= routed have no part (idx null: all have one)
 };
 
 __global__ void __launch_bounds__(128) moe_combine_kernel(CombineDev d) {
@@ -340,7 +357,7 @@ __global__ void __launch_bounds__(128) moe_combine_kernel(CombineDev d) {
     for (int c = threadIdx.x; c < d.width; c += blockDim.x) {
       float acc = d.addend ? ld_as_float(d.addend, d.addend_dt, r * d.ld_addend + c) : 0.f;
       for (int k = 0; k < d.top; ++k)
-        acc = fmaf(d.weight[r * d.top + k], ld_as_float(d.part, d.part_dt, static_cast<long long>(d.inv[r * d.top + k]) * d.ld_part + c), acc);
+        if (!d.idx || d.idx[r * d.top + k] < d.routed) acc = fmaf(d.weight[r * d.top + k], ld_as_float(d.part, d.part_dt, static_cast<long long>(d.inv[r * d.top + k]) * d.ld_part + c), acc);
       st_from_float(d.out, d.out_dt, r * d.ld_out + c, acc);
     }
   }
@@ -417,6 +434,10 @@ extern "C" int vy_moe_route(const VyMoeRoute* p) {
   d.logits = p->logits; d.ld = p->ld_logits; d.scale = p->scale;
   d.idx = p->idx; d.weight = p->weight; d.dense = p->dense;
   d.kind = p->kind; d.raw = p->raw_weights;
+  d.corr = p->correction; d.corr_dt = p->correction_dtype;
+  d.identity = p->identity; d.ident = p->ident;
+  VY_CHECK_ARG((!p->correction || dtype_ok(p->correction_dtype)) && p->identity >= 0 && p->identity < p->experts && (p->identity == 0 || p->ident),
+               "vy_moe_route: bad correction or identity experts (%d of %d)", p->identity, p->experts);
   d.groups = p->groups > 1 ? p->groups : 0; d.keep_groups = d.groups ? p->keep_groups : 0;
   VY_CHECK_ARG(p->kind == VY_ROUTE_SIGMOID || p->kind == VY_ROUTE_SOFTMAX, "vy_moe_route: unknown kind %d", p->kind);
   VY_CHECK_ARG(d.groups == 0 || (p->experts % d.groups == 0 && d.keep_groups > 0 && d.keep_groups <= d.groups &&
@@ -501,6 +522,7 @@ extern "C" int vy_moe_combine(const VyMoeCombine* p) {
   d.part = p->part; d.ld_part = p->ld_part; d.part_dt = p->part_dtype;
   d.addend = p->addend; d.ld_addend = p->ld_addend; d.addend_dt = p->addend_dtype;
   d.out = p->out; d.ld_out = p->ld_out; d.out_dt = p->out_dtype;
+  d.idx = p->idx; d.routed = p->routed;
   const long long blocks = p->rows < 65536 ? p->rows : 65536;
   VY_CUDA_OK(launch_kernel(moe_combine_kernel, dim3(static_cast<unsigned>(blocks)), dim3(128), 0, static_cast<cudaStream_t>(p->stream), d));
   VY_LAUNCH_OK();

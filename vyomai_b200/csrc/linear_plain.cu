@@ -185,7 +185,77 @@ __global__ void __launch_bounds__(128) embed_rows_kernel(int rows, int width, in
                   ok ? scale * ld_as_float(table, table_dt, static_cast<long long>(id) * ld_table + c) : 0.f);
 }
 
+struct PairDev {
+  const int* cu; const int* pos0; const int* slot; const int* ids;
+  int width, vocab, table_dt;
+  const void* table; long long ld_table; const void* pairs; long long ld_pairs;
+  float scale;
+  long long mul_prev, mul_cur; int buckets;   // multipliers reduced modulo buckets by the host: the products fit 64 bits
+  int* prev;
+  void* out; long long ld_out; int out_dt;
+};
+
+// blockIdx.x = token of the portion, blockIdx.y = sequence. Only the portion's first token's CTA touches the sequence's prev_state: it
+// reads the token before the portion and leaves the portion's last one
+__global__ void __launch_bounds__(128) pair_embed_kernel(PairDev d) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ int prev_s;
+  const int s = blockIdx.y;
+  const int base = d.cu[s], n = d.cu[s + 1] - base;
+  for (int i = blockIdx.x; i < n; i += gridDim.x) {
+    const int r = base + i, id = d.ids[r], pos = d.pos0[s] + i;
+    int prev = 0;
+    if (i > 0) prev = d.ids[r - 1];
+    else {
+      if (threadIdx.x == 0) {
+        int* st = d.prev + d.slot[s];
+        prev_s = pos > 0 ? *st : 0;
+        *st = d.ids[base + n - 1];
+      }
+      __syncthreads();
+      prev = prev_s;
+    }
+    long long b = d.buckets;
+    if (pos > 0) {
+      b = (prev * d.mul_prev + id * d.mul_cur) % d.buckets;
+      if (b < 0) b += d.buckets;   // ids below zero
+    }
+    const bool ok = id >= 0 && id < d.vocab;
+    for (int c = threadIdx.x; c < d.width; c += blockDim.x) {
+      const float e = ok ? d.scale * ld_as_float(d.table, d.table_dt, static_cast<long long>(id) * d.ld_table + c) : 0.f;
+      st_from_float(d.out, d.out_dt, static_cast<long long>(r) * d.ld_out + c, e + ld_as_float(d.pairs, d.table_dt, b * d.ld_pairs + c));
+    }
+  }
+}
+
 }  // namespace vy
+
+extern "C" int vy_pair_embed(const VyPairEmbed* p) {
+  using namespace vy;
+  VY_CHECK_ARG(p != nullptr, "vy_pair_embed: null params");
+  if (!vy_device_ok()) {
+    set_error("vy_pair_embed: no sm_100 device (there is no CPU fallback)");
+    return VY_ERR_NO_DEVICE;
+  }
+  VY_CHECK_ARG(p->n_seqs > 0 && p->n_seqs <= 65535 && p->max_new > 0 && p->cu_tokens && p->pos0 && p->slot && p->ids, "vy_pair_embed: bad batch");
+  VY_CHECK_ARG(p->width > 0 && p->vocab > 0 && p->table && p->pairs && p->prev_state && p->out && dtype_ok(p->table_dtype) && dtype_ok(p->out_dtype),
+               "vy_pair_embed: bad tensors");
+  VY_CHECK_ARG(p->buckets > 0 && p->mul_prev >= 0 && p->mul_cur >= 0, "vy_pair_embed: %d buckets and the multipliers must be positive", p->buckets);
+  PairDev d;
+  d.cu = p->cu_tokens; d.pos0 = p->pos0; d.slot = p->slot; d.ids = p->ids;
+  d.width = p->width; d.vocab = p->vocab; d.table_dt = p->table_dtype;
+  d.table = p->table; d.ld_table = p->ld_table; d.pairs = p->pairs; d.ld_pairs = p->ld_pairs;
+  d.scale = p->scale;
+  d.mul_prev = p->mul_prev % p->buckets; d.mul_cur = p->mul_cur % p->buckets; d.buckets = p->buckets;
+  d.prev = p->prev_state;
+  d.out = p->out; d.ld_out = p->ld_out; d.out_dt = p->out_dtype;
+  const unsigned gx = static_cast<unsigned>(p->max_new < 65535 ? p->max_new : 65535);
+  VY_CUDA_OK(launch_kernel(pair_embed_kernel, dim3(gx, p->n_seqs), dim3(128), 0, static_cast<cudaStream_t>(p->stream), d));
+  VY_LAUNCH_OK();
+  count_launch();
+  return VY_OK;
+}
 
 extern "C" int vy_linear_plain(const VyLinear* p) {
   using namespace vy;

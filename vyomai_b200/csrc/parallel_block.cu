@@ -103,14 +103,16 @@ struct GluDev {
   const float* dense; long long ld_dense;
   float limit, shared_limit, alpha;
   void* out; long long ld_out; int out_dt;
+  int interleaved; float shift;   // gate / up columns alternate; the up factor is u + shift
+  const float* sg; long long ld_sg;   // the shared block's weight is its sigmoid (null: 1)
 };
 
-__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float alpha) {
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float alpha, float shift) {
   if (limit > 0.f) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
   }
-  return g * sigmoidf_(alpha * g) * (u + 1.f);
+  return g * sigmoidf_(alpha * g) * (u + shift);
 }
 
 // blockIdx.x = token, threads (and blockIdx.y) over output columns. VEC: 8 adjacent columns per thread with 16 / 32-byte accesses
@@ -121,6 +123,8 @@ __global__ void __launch_bounds__(256) moe_glu_kernel(GluDev d) {
   pdl_wait();
   const long long r = blockIdx.x;
   const int ecols = d.experts * d.ff, cols = ecols + d.shared_ff;
+  const float shared_w = d.sg && d.shared_ff ? sigmoidf_(d.sg[r * d.ld_sg]) : 1.f;
+  const int up = d.interleaved ? 1 : 0, step = d.interleaved ? 2 : 1;   // offset of up_j from gate_j (interleaved), column step
   if (VEC) {
     for (int c0 = (blockIdx.y * 256 + threadIdx.x) * 8; c0 < cols; c0 += gridDim.y * 256 * 8) {
       float y[8];
@@ -128,15 +132,23 @@ __global__ void __launch_bounds__(256) moe_glu_kernel(GluDev d) {
       const int e = routed ? c0 / d.ff : d.experts;
       const int j = routed ? c0 - e * d.ff : c0 - ecols;
       const int half = routed ? d.ff : d.shared_ff;
-      const float w = routed ? (d.dense ? d.dense[r * d.ld_dense + e] : 1.f) : 1.f;
+      const float w = routed ? (d.dense ? d.dense[r * d.ld_dense + e] : 1.f) : shared_w;
       if (w != 0.f) {
         const long long o = r * d.ldh + static_cast<long long>(e) * 2 * d.ff + j;   // the shared block follows the experts' 2 ff columns each
         float g[8], u[8];
-        ld8_as_float(d.h, d.h_dt, o, g);
-        ld8_as_float(d.h, d.h_dt, o + half, u);
+        if (d.interleaved) {
+          float p[16];
+          ld8_as_float(d.h, d.h_dt, o + j, *reinterpret_cast<float (*)[8]>(p));
+          ld8_as_float(d.h, d.h_dt, o + j + 8, *reinterpret_cast<float (*)[8]>(p + 8));
+#pragma unroll
+          for (int k = 0; k < 8; ++k) { g[k] = p[2 * k]; u[k] = p[2 * k + 1]; }
+        } else {
+          ld8_as_float(d.h, d.h_dt, o, g);
+          ld8_as_float(d.h, d.h_dt, o + half, u);
+        }
         const float lim = routed ? d.limit : d.shared_limit;
 #pragma unroll
-        for (int k = 0; k < 8; ++k) y[k] = w * clamped_glu(g[k], u[k], lim, d.alpha);
+        for (int k = 0; k < 8; ++k) y[k] = w * clamped_glu(g[k], u[k], lim, d.alpha, d.shift);
       } else {
 #pragma unroll
         for (int k = 0; k < 8; ++k) y[k] = 0.f;
@@ -151,13 +163,13 @@ __global__ void __launch_bounds__(256) moe_glu_kernel(GluDev d) {
       const int e = c / d.ff, j = c - e * d.ff;
       const float w = d.dense ? d.dense[r * d.ld_dense + e] : 1.f;
       if (w != 0.f) {
-        const long long o = r * d.ldh + static_cast<long long>(e) * 2 * d.ff + j;
-        y = w * clamped_glu(ld_as_float(d.h, d.h_dt, o), ld_as_float(d.h, d.h_dt, o + d.ff), d.limit, d.alpha);
+        const long long o = r * d.ldh + static_cast<long long>(e) * 2 * d.ff + step * j;
+        y = w * clamped_glu(ld_as_float(d.h, d.h_dt, o), ld_as_float(d.h, d.h_dt, o + (up ? 1 : d.ff)), d.limit, d.alpha, d.shift);
       }
     } else {
       const int j = c - ecols;
-      const long long o = r * d.ldh + static_cast<long long>(d.experts) * 2 * d.ff + j;
-      y = clamped_glu(ld_as_float(d.h, d.h_dt, o), ld_as_float(d.h, d.h_dt, o + d.shared_ff), d.shared_limit, d.alpha);
+      const long long o = r * d.ldh + static_cast<long long>(d.experts) * 2 * d.ff + step * j;
+      y = shared_w * clamped_glu(ld_as_float(d.h, d.h_dt, o), ld_as_float(d.h, d.h_dt, o + (up ? 1 : d.shared_ff)), d.shared_limit, d.alpha, d.shift);
     }
     st_from_float(d.out, d.out_dt, r * d.ld_out + c, y);
   }
@@ -226,6 +238,7 @@ struct RopeHeadsDev {
   float eps, rot_scale, q_scale, k_scale;
   void* k_out; long long ld_k_out;
   const void* q_norm; const void* k_norm; int norm_dt;   // RMS norm with a weight [dim] before the rotation; null: none
+  float q_temp; int q_temp_every;   // > 0: queries times 1 + q_temp ln(floor((pos + 1) / every) + 1)
 };
 
 __global__ void __launch_bounds__(256, 4) rope_heads_kernel(RopeHeadsDev d) {
@@ -302,6 +315,7 @@ __global__ void __launch_bounds__(256, 4) rope_heads_kernel(RopeHeadsDev d) {
 #pragma unroll
       for (int r = 0; r < 8; ++r) ss = fmaf(ps[r], ps[r], ss);
       float f = is_q ? d.q_scale : d.k_scale;
+      if (is_q && d.q_temp_every > 0) f *= fmaf(d.q_temp, logf(static_cast<float>((pos + 1) / d.q_temp_every) + 1.f), 1.f);
       if (d.unit_rms) f /= sqrtf(warp_sum(ss) / static_cast<float>(b.dim) + d.eps);
       void* dst;
       long long dof;
@@ -418,6 +432,8 @@ extern "C" int vy_moe_glu(const VyMoeGlu* p) {
   d.h = p->h; d.ldh = p->ldh; d.h_dt = p->h_dtype;
   d.dense = p->dense; d.ld_dense = p->ld_dense;
   d.limit = p->limit; d.shared_limit = p->shared_limit; d.alpha = p->alpha;
+  d.interleaved = p->interleaved ? 1 : 0; d.shift = p->no_shift ? 0.f : 1.f;
+  d.sg = p->shared_gate; d.ld_sg = p->ld_gate;
   d.out = p->out; d.ld_out = p->ld_out; d.out_dt = p->out_dtype;
   const int cols = d.experts * d.ff + d.shared_ff;
   const auto al = [](const void* q, size_t n) { return reinterpret_cast<uintptr_t>(q) % n == 0; };
@@ -455,7 +471,7 @@ extern "C" int vy_rope_kv_write(const VyRopeKvWrite* p) {
   d.kp = p->k_pool; d.vp = paged ? p->v_pool : nullptr; d.pool_dt = p->pool_dtype;
   const unsigned gx = static_cast<unsigned>(p->max_new < 65535 ? p->max_new : 65535);
   const bool general = !paged || p->half_layout || p->unit_rms || (p->rot_scale != 0.f && p->rot_scale != 1.f) || (p->q_scale != 0.f && p->q_scale != 1.f) ||
-                       (p->k_scale != 0.f && p->k_scale != 1.f) || p->q_norm || p->k_norm;
+                       (p->k_scale != 0.f && p->k_scale != 1.f) || p->q_norm || p->k_norm || p->q_temp_every > 0;
   if (general) {
     VY_CHECK_ARG((!p->q_norm && !p->k_norm) || (dtype_ok(p->norm_dtype) && !p->unit_rms), "vy_rope_kv_write: a weighted norm before the rotation excludes unit_rms after it");
     VY_CHECK_ARG(p->dim <= 256, "vy_rope_kv_write: dim %d > 256", p->dim);
@@ -468,6 +484,7 @@ extern "C" int vy_rope_kv_write(const VyRopeKvWrite* p) {
     g.k_scale = p->k_scale == 0.f ? 1.f : p->k_scale;
     g.k_out = p->k_out; g.ld_k_out = p->ld_k_out;
     g.q_norm = p->q_norm; g.k_norm = p->k_norm; g.norm_dt = p->norm_dtype;
+    g.q_temp = p->q_temp; g.q_temp_every = p->q_temp_every;
     // single tokens: a warp per head in flight (up to 8), few CTAs; prompts: 4 warps per token, more CTAs per SM (measured: 8 warps cost
     // prompts 0.23 -> 0.34 ms over 4 launches of 8192 tokens and saved single-token steps 29 -> 21 us)
     const int units = p->heads + p->kv_heads;

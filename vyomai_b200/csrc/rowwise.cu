@@ -59,6 +59,8 @@ struct SandDev {
   const int* row_index;
   const float* x; long long ldx; const float* y; long long ldy;
   const void* w1; const void* b1; const void* w2; const void* b2; int w_dt;
+  int kind;   // VY_CLOSE_LAYER, or RMS norms with the weight as it is / stored around zero
+  const void* u; long long ld_u; int u_dt; const float* u_coef;   // y + u_coef[row] * u is what is normed (u null: y)
   float eps;
   float* xo; long long ld_xo;
   void* copy; long long ld_copy; int copy_dt;
@@ -80,14 +82,18 @@ __device__ __forceinline__ float row_sum(float v, float* part, int lr, int lt) {
   return v;
 }
 
-// v <- layer norm of the row's values (entries past the width stay out of the statistics)
+// v <- layer norm (or RMS norm, d.kind) of the row's values (entries past the width stay out of the statistics)
 template <int TPR, int NC, bool VEC>
 __device__ __forceinline__ void norm_row(float (&v)[NC], const SandDev& d, const void* w, const void* b, float* part, int lr, int lt) {
   auto col = [&](int i) { return VEC ? 4 * lt + (i >> 2) * 4 * TPR + (i & 3) : lt + i * TPR; };
-  float s = 0.f;
+  float mean = 0.f;
+  if (d.kind == VY_CLOSE_LAYER) {
+    float s = 0.f;
 #pragma unroll
-  for (int i = 0; i < NC; ++i) s += v[i];
-  const float mean = row_sum<TPR>(s, part, lr, lt) / static_cast<float>(d.width);
+    for (int i = 0; i < NC; ++i) s += v[i];
+    mean = row_sum<TPR>(s, part, lr, lt) / static_cast<float>(d.width);
+  }
+  const float w_add = d.kind == VY_CLOSE_RMS_CENTRED ? 1.f : 0.f;
   float q = 0.f;
 #pragma unroll
   for (int i = 0; i < NC; ++i) {
@@ -110,13 +116,28 @@ __device__ __forceinline__ void norm_row(float (&v)[NC], const SandDev& d, const
       v[i + 2] = fmaf(v[i + 2] * inv, w1.x, b1.x);
       v[i + 3] = fmaf(v[i + 3] * inv, w1.y, b1.y);
     }
+  } else if (VEC && d.w_dt == VY_BF16 && w) {
+#pragma unroll
+    for (int i = 0; i < NC; i += 4) {
+      if (col(i) >= d.width) continue;
+      const uint2 wr = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(w) + col(i));
+      const __nv_bfloat162* wp = reinterpret_cast<const __nv_bfloat162*>(&wr);
+      const float2 w0 = __bfloat1622float2(wp[0]), w1 = __bfloat1622float2(wp[1]);
+      v[i] *= inv * (w_add + w0.x);
+      v[i + 1] *= inv * (w_add + w0.y);
+      v[i + 2] *= inv * (w_add + w1.x);
+      v[i + 3] *= inv * (w_add + w1.y);
+      if (b)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[i + e] += ld_as_float(b, d.w_dt, col(i) + e);
+    }
   } else {
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
       const int c = col(i);
       if (c >= d.width) continue;
       float z = v[i] * inv;
-      if (w) z *= ld_as_float(w, d.w_dt, c);
+      if (w) z *= w_add + ld_as_float(w, d.w_dt, c);
       if (b) z += ld_as_float(b, d.w_dt, c);
       v[i] = z;
     }
@@ -175,6 +196,16 @@ __global__ void __launch_bounds__(TPR < 256 ? 256 : TPR) sandwich_norm_kernel(Sa
   load(d.x + st * d.ldx, xv);
   if (d.y) {
     load(d.y + st * d.ldy, yv);
+    if (d.u) {
+      const float uc = live ? d.u_coef[st] : 0.f;
+      if (uc != 0.f) {   // a zero weight leaves the row unread
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+          const int c = VEC ? 4 * lt + (i >> 2) * 4 * TPR + (i & 3) : lt + i * TPR;
+          if (c < d.width) yv[i] = fmaf(uc, ld_as_float(d.u, d.u_dt, st * d.ld_u + c), yv[i]);
+        }
+      }
+    }
     norm_row<TPR, NC, VEC>(yv, d, d.w1, d.b1, part, lr, lt);
 #pragma unroll
     for (int i = 0; i < NC; ++i) xv[i] += yv[i];
@@ -270,6 +301,11 @@ extern "C" int vy_sandwich_norm(const VySandwichNorm* p) {
   d.rows = p->rows; d.width = p->width; d.row_index = p->row_index;
   d.x = p->x; d.ldx = p->ldx; d.y = p->y; d.ldy = p->ldy;
   d.w1 = p->w1; d.b1 = p->b1; d.w2 = p->w2; d.b2 = p->b2; d.w_dt = p->w_dtype; d.eps = p->eps;
+  VY_CHECK_ARG(p->norm_kind >= VY_CLOSE_LAYER && p->norm_kind <= VY_CLOSE_RMS_CENTRED && (p->norm_kind == VY_CLOSE_LAYER || (!p->b1 && !p->b2)),
+               "vy_sandwich_norm: norm kind %d (RMS norms take no bias)", p->norm_kind);
+  VY_CHECK_ARG(!p->u || (p->y && p->u_coef && dtype_ok(p->u_dtype)), "vy_sandwich_norm: a second result needs the first, its dtype and its weights");
+  d.kind = p->norm_kind;
+  d.u = p->u; d.ld_u = p->ld_u; d.u_dt = p->u_dtype; d.u_coef = p->u_coef;
   d.xo = p->x_out; d.ld_xo = p->ld_x_out;
   d.copy = p->copy; d.ld_copy = p->ld_copy; d.copy_dt = p->copy_dtype;
   d.out = p->out; d.ld_out = p->ld_out; d.out_dt = p->out_dtype;

@@ -56,15 +56,15 @@ __global__ void __launch_bounds__(128) rms_norm_kernel(NormDev d) {
 }
 
 // The same with the row held in registers (one read of x) and TPR threads per row, 256 threads per CTA: for widths up to
-// 8 TPR. Few wide rows (single-token steps) get many threads each; many narrow rows get a warp each.
+// NC TPR. Few wide rows (single-token steps) get many threads each; many narrow rows get a warp each.
 // VEC: x, gate and out rows start on 16-byte boundaries (out: 8 when bf16) and the width is a multiple of 4, x and gate are fp32,
 // and an accumulating call's out is fp32: each thread then moves two groups of 4 adjacent elements instead of 8 strided ones,
 // a quarter of the load / store / address instructions (a single-token call is one short dependent instruction stream per warp)
-template <int TPR, bool VEC>
+template <int TPR, bool VEC, int NC = 8>
 __global__ void __launch_bounds__(256) rms_norm_cached_kernel(NormDev d) {
   pdl_trigger();
   pdl_wait();
-  constexpr int NC = 8, RPB = 256 / TPR;
+  constexpr int RPB = 256 / TPR;
   __shared__ float part[RPB][TPR / 32 + 1];
   const int lr = threadIdx.x / TPR, lt = threadIdx.x % TPR;
   const unsigned r = blockIdx.x * static_cast<unsigned>(RPB) + lr;   // the launcher keeps rows below 2^31: 32-bit division
@@ -240,6 +240,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(WinDev d) {
   visible_keys(d, pos, nA, lowB);
   const int count = nA + (pos + 1 - lowB);
   const float sc_mul = head_scale_of(d, h), sc_add = head_bias_of(d, h);
+  const float slope = head_slope_of(d, h), two_over_cap = d.softcap > 0.f ? 2.f / d.softcap : 0.f;
   float m = -INFINITY, l = SIG ? 1.f : 0.f;
   if (!SIG && d.sink) {
     m = ld_as_float(d.sink, d.sink_dt, h);
@@ -260,6 +261,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(WinDev d) {
       const int kp = c < nA ? c : lowB + (c - nA);
       row = static_cast<long long>(tab[kp / d.bs]) * d.bs + kp % d.bs;
       sc = dot_row(d.kp, d.pool_dt, row * kstride + static_cast<long long>(g) * d.dim, d.dim, qs) * sc_mul + sc_add;
+      sc = shaped_score(d, sc, two_over_cap, slope, pos - kp);
     }
     float p;
     if constexpr (SIG) {
@@ -345,14 +347,17 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(WinDe
   }
   const int* tab = d.table + static_cast<long long>(s) * d.tw;
   const long long kstride = d.k_row, vstride = d.v_row;
+  const float two_over_cap = d.softcap > 0.f ? 2.f / d.softcap : 0.f;
   for (int c0 = WD_KEYS * warp; c0 < count; c0 += WD_KEYS * WD_WARPS) {
     long long row[WD_KEYS];
+    int dist[WD_KEYS];
     float sc[HG][WD_KEYS], vv[WD_KEYS][WA_VR];
 #pragma unroll
     for (int u = 0; u < WD_KEYS; ++u) {
       const int c = min(c0 + u, count - 1);   // past the end: a repeat of the last key, given weight 0 below
       const int kp = c < nA ? c : lowB + (c - nA);
       row[u] = static_cast<long long>(tab[kp / d.bs]) * d.bs + kp % d.bs;
+      dist[u] = pos - kp;
 #pragma unroll
       for (int hh = 0; hh < HG; ++hh) sc[hh][u] = 0.f;
     }
@@ -407,11 +412,11 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(WinDe
     }
 #pragma unroll
     for (int hh = 0; hh < HG; ++hh) {
-      const float sc_add = head_bias_of(d, h0 + hh);
+      const float sc_add = head_bias_of(d, h0 + hh), slope = head_slope_of(d, h0 + hh);
       if constexpr (SIG) {
         float p[WD_KEYS];
 #pragma unroll
-        for (int u = 0; u < WD_KEYS; ++u) p[u] = c0 + u < count ? sigmoidf_(warp_sum(sc[hh][u]) + sc_add) : 0.f;
+        for (int u = 0; u < WD_KEYS; ++u) p[u] = c0 + u < count ? sigmoidf_(shaped_score(d, warp_sum(sc[hh][u]) + sc_add, two_over_cap, slope, dist[u])) : 0.f;
 #pragma unroll
         for (int r = 0; r < WA_VR; ++r)
 #pragma unroll
@@ -421,7 +426,7 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(WinDe
       float m_new = m[hh];
 #pragma unroll
       for (int u = 0; u < WD_KEYS; ++u) {
-        sc[hh][u] = c0 + u < count ? warp_sum(sc[hh][u]) + sc_add : -INFINITY;
+        sc[hh][u] = c0 + u < count ? shaped_score(d, warp_sum(sc[hh][u]) + sc_add, two_over_cap, slope, dist[u]) : -INFINITY;
         m_new = fmaxf(m_new, sc[hh][u]);
       }
       const float corr = m[hh] == -INFINITY ? 0.f : expf(m[hh] - m_new);
@@ -853,7 +858,7 @@ extern "C" int vy_rms_norm(const VyRmsNorm* p) {
   VY_CHECK_ARG(!p->copy || (dtype_ok(p->copy_dtype) && p->out_dtype == VY_F32), "vy_rms_norm: the second copy goes with an fp32 out");
   d.copy = p->copy; d.ld_copy = p->ld_copy; d.copy_dt = p->copy_dtype;
   cudaStream_t st = static_cast<cudaStream_t>(p->stream);
-  const int tpr = d.width <= 256 ? 32 : d.width <= 1024 ? 128 : d.width <= 2048 ? 256 : 0;
+  const int tpr = d.width <= 256 ? 32 : d.width <= 1024 ? 128 : d.width <= 8192 ? 256 : 0;
   const long long blocks = tpr ? (d.rows + 256 / tpr - 1) / (256 / tpr) : (d.rows + 3) / 4;
   VY_CHECK_ARG(blocks <= 2147483647LL && d.rows <= 2147483647LL, "vy_rms_norm: too many rows");
   const dim3 grid(static_cast<unsigned>(blocks));
@@ -865,6 +870,8 @@ extern "C" int vy_rms_norm(const VyRmsNorm* p) {
                                 : launch_kernel(rms_norm_cached_kernel<32, false>, grid, dim3(256), 0, st, d));
   else if (tpr == 128) VY_CUDA_OK(vec ? launch_kernel(rms_norm_cached_kernel<128, true>, grid, dim3(256), 0, st, d)
                                       : launch_kernel(rms_norm_cached_kernel<128, false>, grid, dim3(256), 0, st, d));
+  else if (tpr == 256 && d.width > 2048) VY_CUDA_OK(vec ? launch_kernel(rms_norm_cached_kernel<256, true, 32>, grid, dim3(256), 0, st, d)
+                                                        : launch_kernel(rms_norm_cached_kernel<256, false, 32>, grid, dim3(256), 0, st, d));
   else if (tpr == 256) VY_CUDA_OK(vec ? launch_kernel(rms_norm_cached_kernel<256, true>, grid, dim3(256), 0, st, d)
                                       : launch_kernel(rms_norm_cached_kernel<256, false>, grid, dim3(256), 0, st, d));
   else VY_CUDA_OK(launch_kernel(rms_norm_kernel, grid, dim3(128), 0, st, d));
@@ -929,6 +936,8 @@ extern "C" int vy_window_attn(const VyWinAttn* p) {
   VY_CHECK_ARG(p->weight_kind == VY_ATTN_SOFTMAX || (p->weight_kind == VY_ATTN_SIGMOID && !p->sink), "vy_window_attn: weight kind %d (sigmoid weights take no sink)", p->weight_kind);
   d.sigmoid = p->weight_kind == VY_ATTN_SIGMOID ? 1 : 0;
   d.head_scale = p->head_scale; d.head_bias = p->head_bias;
+  VY_CHECK_ARG(p->softcap >= 0.f, "vy_window_attn: negative softcap");
+  d.softcap = p->softcap; d.head_slope = p->head_slope;
   d.gate = p->gate; d.ld_gate = p->ld_gate; d.gate_dt = p->gate_dtype;
   d.out = p->out; d.ld_out = p->ld_out; d.out_dt = p->out_dtype;
   cudaStream_t st = static_cast<cudaStream_t>(p->stream);

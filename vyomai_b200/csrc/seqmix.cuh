@@ -19,6 +19,7 @@ __device__ __forceinline__ float apply_uact(float x, int act) {
     default: return x;
   }
 }
+constexpr float MIN_LOG_DECAY = -1e4f;   // exp of it is 0 in fp32; keeps sums and differences of log decays finite
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -28,6 +29,12 @@ __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
   return v;
+}
+
+// cap * tanh(s / cap) as cap * (1 - 2 / (1 + e^(2 s / cap))): expf and a fast reciprocal, absolute error a few 1e-7 * cap (the softmax
+// that follows depends on score differences, i.e. on absolute error); e^x overflowing to inf gives exactly cap, underflow exactly -cap
+__device__ __forceinline__ float cap_score(float s, float cap, float two_over_cap) {
+  return cap > 0.f ? cap * (1.f - __fdividef(2.f, 1.f + expf(s * two_over_cap))) : s;
 }
 
 __device__ __forceinline__ float dot4(const float4 a, const float4 b, float acc) {
@@ -120,10 +127,17 @@ struct WinDev {
   void* out; long long ld_out; int out_dt;
   int sigmoid;   // the weight of a visible key is sigmoid(score), not normalised over the keys
   const float* head_scale; const float* head_bias;   // score = (q . k) * scale * head_scale[h] + head_bias[h]; null: 1 / 0
+  float softcap; const float* head_slope;   // then: cap tanh(score / cap) (cap > 0), minus head_slope[h] * distance (null: 0)
 };
 
 __device__ __forceinline__ float head_scale_of(const WinDev& d, int h) { return d.head_scale ? d.scale * d.head_scale[h] : d.scale; }
 __device__ __forceinline__ float head_bias_of(const WinDev& d, int h) { return d.head_bias ? d.head_bias[h] : 0.f; }
+
+__device__ __forceinline__ float head_slope_of(const WinDev& d, int h) { return d.head_slope ? d.head_slope[h] : 0.f; }
+// the capped score minus the distance's share; two_over_cap = 2 / softcap
+__device__ __forceinline__ float shaped_score(const WinDev& d, float z, float two_over_cap, float slope, int distance) {
+  return fmaf(-slope, static_cast<float>(distance), cap_score(z, d.softcap, two_over_cap));
+}
 
 // One query's visible keys at position pos: [0, nA) (kept first tokens) and [lowB, pos] (the window, or the query's chunk), disjoint
 __device__ __forceinline__ void visible_keys(const WinDev& d, int pos, int& nA, int& lowB) {
@@ -143,6 +157,10 @@ struct RecDev {
   int heads, kv_heads, dim, vdim;
   float unit_eps;
   int prepared;   // delta rule: q / k are unit vectors already (q scaled), `a` holds the decays and `b` the write strengths
+  // chunked form with a decay and a write strength per head and token (state-space recurrence): strength w = softplus(dt + dt_bias[h]),
+  // decay exp(-exp(a_log[h]) w), plus skip[h] v in the output, the whole times gate_act(gate); dt_bias, a_log, skip share a_log_dt
+  const float* dt; long long ld_dt; const void* dt_bias; const void* skip;
+  const float* gate; long long ld_gate; int gate_act;
   float q_scale;  // gated linear attention (the delta kernel without its correction term): multiplies q as it is read
   float* state;
   void* out; long long ld_out; int out_dt;
@@ -150,6 +168,7 @@ struct RecDev {
 
 // Prompt-sized steps: defined in seqmix_tiled.cu.
 cudaError_t launch_linear_attn_chunked(const RecDev& d, int n_seqs, cudaStream_t st);
+cudaError_t launch_ssd_chunked(const RecDev& d, int n_seqs, cudaStream_t st);
 cudaError_t launch_window_attn_tiled(const WinDev& d, int n_seqs, int max_new, cudaStream_t st);
 // Single tokens whose query heads share key / value rows in groups of 8 or more (latent rows): heads as the rows of a tile.
 bool window_attn_heads_applies(const WinDev& d);

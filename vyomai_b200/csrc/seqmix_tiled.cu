@@ -4,7 +4,9 @@
 //   * linear attention with a fixed decay, chunk by chunk: for a chunk of C tokens with the state S0 before it,
 //       O = (Q K^T . D) V + diag(decay^(i+1)) Q S0,   D[i][j] = decay^(i-j) for j <= i, else 0
 //       S = decay^C S0 + sum_j decay^(C-1-j) k_j v_j^T
-//     one CTA owns (sequence, head, 64 value columns) and walks the chunks in order with its slice of S in shared memory;
+//     one CTA owns (sequence, head, 64 value columns) and walks the chunks in order with its slice of S in shared memory.
+//     The state-space recurrence runs on the same kernel with a decay and a write strength per token: decay^(i-j) becomes
+//     exp(L_i - L_j) w_j with L the summed log decays of the chunk (kept as two floats: their differences are what counts);
 //   * windowed softmax attention with kept first tokens and a sink over pages: one CTA owns 64 queries of one head, walks
 //     the visible keys in tiles of 64 (the kept prefix first, then the window band) with an online softmax.
 //
@@ -20,11 +22,11 @@ constexpr int LA_C = 64;    // tokens per chunk
 constexpr int LA_T = 256;   // threads: a 16 x 16 grid; thread (ti, tj) owns rows ti + 16 r and VS / 16 adjacent value columns
 constexpr int LA_LDP = LA_C + 4;
 
-template <int DP, int VS>   // VS: value columns per CTA, 32 (two CTAs per SM, more CTAs) or 64 (less repeated work)
+template <int DP, int VS, bool TD = false>   // VS: value columns per CTA, 32 (two CTAs per SM, more CTAs) or 64 (less repeated work)
 struct LaSmem {
   static constexpr int LDQ = DP + 4;    // row stride of the q / k chunks (floats): rows 1 apart start in distinct 16-byte bank groups
   static constexpr int LDV = VS + 4;    // row stride of the v chunk and the state slice
-  static constexpr int floats = 2 * LA_C * LDQ + LA_C * LDV + LA_C * LA_LDP + DP * LDV + LA_C + 4;
+  static constexpr int floats = 2 * LA_C * LDQ + LA_C * LDV + LA_C * LA_LDP + DP * LDV + (TD ? 5 * LA_C + 4 : LA_C + 4);
 };
 
 template <int NV>
@@ -43,11 +45,12 @@ __device__ __forceinline__ void axpyv(float (&acc)[NV], const float a, const flo
   for (int e = 0; e < NV; ++e) acc[e] = fmaf(a, x[e], acc[e]);
 }
 
-template <int DP, int VS, int OCC>   // OCC: CTAs per SM the register budget is set for
+// OCC: CTAs per SM the register budget is set for; TD: decay and write strength per token (q, k shared by groups of heads)
+template <int DP, int VS, int OCC, bool TD>
 __global__ void __launch_bounds__(LA_T, OCC) linear_attn_chunk_kernel(RecDev d, bool vec) {
   pdl_trigger();
   pdl_wait();
-  constexpr int LDQ = LaSmem<DP, VS>::LDQ, LDV = LaSmem<DP, VS>::LDV, LDP = LA_LDP;
+  constexpr int LDQ = LaSmem<DP, VS, TD>::LDQ, LDV = LaSmem<DP, VS, TD>::LDV, LDP = LA_LDP;
   constexpr int NV = VS / 16;               // value columns per thread
   constexpr int DR = DP / 16;               // state rows per thread in the update
   extern __shared__ __align__(16) float la_smem[];
@@ -57,11 +60,23 @@ __global__ void __launch_bounds__(LA_T, OCC) linear_attn_chunk_kernel(RecDev d, 
   float* Ps = Vs + LA_C * LDV;              // [C][LDP]
   float* Ss = Ps + LA_C * LDP;              // [DP][LDV]
   float* pw = Ss + DP * LDV;                // decay^n, n = 0 .. C
+  // TD: per token of the chunk the summed log decays (high and low part), the write strength, e^L and e^(L_end - L) times the strength
+  float* Lh = pw + 4;
+  float* Ll = Lh + LA_C;
+  float* wr = Ll + LA_C;
+  float* eL = wr + LA_C;
+  float* es = eL + LA_C;
   const int s = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * VS;
   const int t = threadIdx.x, ti = t >> 4, tj = t & 15;
   const int base = d.cu[s], n = d.cu[s + 1] - base;
   if (n <= 0) return;
-  if (t <= LA_C) pw[t] = static_cast<float>(pow(static_cast<double>(d.decay[h]), static_cast<double>(t)));
+  const int hq = TD ? h / (d.heads / d.kv_heads) : h;
+  float rate = 0.f, dt_b = 0.f, skip = 0.f;
+  if constexpr (TD) {
+    rate = expf(ld_as_float(d.a_log, d.a_log_dt, h));
+    dt_b = ld_as_float(d.dt_bias, d.a_log_dt, h);
+    skip = ld_as_float(d.skip, d.a_log_dt, h);
+  } else if (t <= LA_C) pw[t] = static_cast<float>(pow(static_cast<double>(d.decay[h]), static_cast<double>(t)));
   float* sp = d.state + (static_cast<long long>(d.slot[s]) * d.heads + h) * d.dim * d.vdim;
   const bool carried = d.pos0[s] > 0;
   for (int e = t; e < DP * VS; e += LA_T) {
@@ -74,11 +89,41 @@ __global__ void __launch_bounds__(LA_T, OCC) linear_attn_chunk_kernel(RecDev d, 
     {
       const long long r0 = base + t0;
       rows_to_smem<LA_T>(Qs, LDQ, LA_C, d.dim, DP, d.q, d.in_dt, vec, d.in_act,
-                         [&](int tt) { return tt < nt ? (r0 + tt) * d.ldq + static_cast<long long>(h) * d.dim : -1LL; });
+                         [&](int tt) { return tt < nt ? (r0 + tt) * d.ldq + static_cast<long long>(hq) * d.dim : -1LL; });
       rows_to_smem<LA_T>(Ks, LDQ, LA_C, d.dim, DP, d.k, d.in_dt, vec, d.in_act,
-                         [&](int tt) { return tt < nt ? (r0 + tt) * d.ldk + static_cast<long long>(h) * d.dim : -1LL; });
+                         [&](int tt) { return tt < nt ? (r0 + tt) * d.ldk + static_cast<long long>(hq) * d.dim : -1LL; });
       rows_to_smem<LA_T>(Vs, LDV, LA_C, min(VS, d.vdim - v0), VS, d.v, d.in_dt, vec, d.in_act,
                          [&](int tt) { return tt < nt ? (r0 + tt) * d.ldv + static_cast<long long>(h) * d.vdim + v0 : -1LL; });
+      if constexpr (TD) {
+        if (t < 32) {   // lane: tokens 2 t, 2 t + 1; tokens past the end neither decay nor write
+          double la[2];
+          float w[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int tt = 2 * t + e;
+            w[e] = tt < nt ? softplusf_(d.dt[(r0 + tt) * d.ld_dt + h] + dt_b) : 0.f;
+            la[e] = fmaxf(-rate * w[e], MIN_LOG_DECAY);
+          }
+          double run = la[0] + la[1];
+#pragma unroll
+          for (int o = 1; o < 32; o <<= 1) {
+            const double x = __shfl_up_sync(0xffffffffu, run, o);
+            if (t >= o) run += x;
+          }
+          const double end = __shfl_sync(0xffffffffu, run, 31);
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const double L = e ? run : run - la[1];
+            const int tt = 2 * t + e;
+            Lh[tt] = static_cast<float>(L);
+            Ll[tt] = static_cast<float>(L - static_cast<double>(Lh[tt]));
+            wr[tt] = w[e];
+            eL[tt] = expf(static_cast<float>(L));
+            es[tt] = expf(static_cast<float>(end - L)) * w[e];
+          }
+          if (t == 0) pw[0] = expf(static_cast<float>(end));
+        }
+      }
     }
     __syncthreads();
     // one pass over the channels feeds both contractions that read the chunk's queries:
@@ -119,7 +164,16 @@ __global__ void __launch_bounds__(LA_T, OCC) linear_attn_chunk_kernel(RecDev d, 
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int i = ti + 16 * r, j = tj + 16 * c;
-        Ps[i * LDP + j] = (c <= r && j <= i && i < nt) ? p[r][c] * pw[i - j] : 0.f;
+        if constexpr (TD) {
+          float x = 0.f;
+          if (c <= r && j <= i && i < nt) {
+            x = p[r][c] * (expf((Lh[i] - Lh[j]) + (Ll[i] - Ll[j])) * wr[j]);
+            if (j == i) x += skip;
+          }
+          Ps[i * LDP + j] = x;
+        } else {
+          Ps[i * LDP + j] = (c <= r && j <= i && i < nt) ? p[r][c] * pw[i - j] : 0.f;
+        }
       }
     __syncthreads();
     // inside the chunk: oa[r][e] = sum_j P[ti + 16 r][j] V[j][NV tj + e]; row block r only sees j < 16 (r + 1)
@@ -153,11 +207,17 @@ __global__ void __launch_bounds__(LA_T, OCC) linear_attn_chunk_kernel(RecDev d, 
     for (int r = 0; r < 4; ++r) {
       const int i = ti + 16 * r;
       if (i < nt) {
-        const float wi = pw[i + 1];
+        const float wi = TD ? eL[i] : pw[i + 1];
         const long long o = static_cast<long long>(base + t0 + i) * d.ld_out + static_cast<long long>(h) * d.vdim + v0 + NV * tj;
 #pragma unroll
         for (int e = 0; e < NV; ++e)
-          if (v0 + NV * tj + e < d.vdim) st_from_float(d.out, d.out_dt, o + e, fmaf(wi, oi[r][e], oa[r][e]));
+          if (v0 + NV * tj + e < d.vdim) {
+            float y = fmaf(wi, oi[r][e], oa[r][e]);
+            if constexpr (TD) {
+              if (d.gate) y *= apply_uact(d.gate[static_cast<long long>(base + t0 + i) * d.ld_gate + static_cast<long long>(h) * d.vdim + v0 + NV * tj + e], d.gate_act);
+            }
+            st_from_float(d.out, d.out_dt, o + e, y);
+          }
       }
     }
     // the state after the chunk: rows ti DR .. ti DR + DR - 1, columns NV tj .. (each thread owns its tile of Ss)
@@ -168,7 +228,7 @@ __global__ void __launch_bounds__(LA_T, OCC) linear_attn_chunk_kernel(RecDev d, 
       for (int e = 0; e < NV; ++e) sa[x][e] = 0.f;
 #pragma unroll 2
     for (int j = 0; j < nt; ++j) {
-      const float w = pw[nt - 1 - j];
+      const float w = TD ? es[j] : pw[nt - 1 - j];
       float vv[NV];
       ldv<NV>(Vs + j * LDV + NV * tj, vv);
 #pragma unroll
@@ -187,7 +247,7 @@ __global__ void __launch_bounds__(LA_T, OCC) linear_attn_chunk_kernel(RecDev d, 
 #pragma unroll
       for (int x = 0; x < DR; ++x) axpyv<NV>(sa[x], kk[x], vv);
     }
-    const float wc = pw[nt];
+    const float wc = TD ? pw[0] : pw[nt];
 #pragma unroll
     for (int x = 0; x < DR; ++x) {
       float* sr = Ss + (ti * DR + x) * LDV + NV * tj;
@@ -202,28 +262,31 @@ __global__ void __launch_bounds__(LA_T, OCC) linear_attn_chunk_kernel(RecDev d, 
   }
 }
 
-template <int DP, int VS, int OCC>
+template <int DP, int VS, int OCC, bool TD = false>
 static cudaError_t launch_la(const RecDev& d, int n_seqs, cudaStream_t st) {
-  constexpr size_t smem = sizeof(float) * LaSmem<DP, VS>::floats;
+  constexpr size_t smem = sizeof(float) * LaSmem<DP, VS, TD>::floats;
   static bool once = false;
   if (!once) {
-    cudaError_t e = cudaFuncSetAttribute(linear_attn_chunk_kernel<DP, VS, OCC>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    cudaError_t e = cudaFuncSetAttribute(linear_attn_chunk_kernel<DP, VS, OCC, TD>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return e;
     once = true;
   }
   const auto al = [](const void* p, long long ld) { return reinterpret_cast<uintptr_t>(p) % 16 == 0 && ld % 4 == 0; };
   const bool vec = d.in_dt == VY_F32 && d.dim % 4 == 0 && d.vdim % 4 == 0 && al(d.q, d.ldq) && al(d.k, d.ldk) && al(d.v, d.ldv);
-  return launch_kernel(linear_attn_chunk_kernel<DP, VS, OCC>, dim3((d.vdim + VS - 1) / VS, d.heads, n_seqs), dim3(LA_T), smem, st, d, vec);
+  return launch_kernel(linear_attn_chunk_kernel<DP, VS, OCC, TD>, dim3((d.vdim + VS - 1) / VS, d.heads, n_seqs), dim3(LA_T), smem, st, d, vec);
 }
 
-template <int DP>
+template <int DP, bool TD = false>
 static cudaError_t launch_la_dp(const RecDev& d, int n_seqs, cudaStream_t st) {
   // 64-column slices repeat the chunk's q k^T half as often; 32-column slices when those would leave SMs without a CTA
   const long long ctas64 = static_cast<long long>((d.vdim + 63) / 64) * d.heads * n_seqs;
-  if (ctas64 >= 148) return launch_la<DP, 64, 1>(d, n_seqs, st);
+  if constexpr (DP > 128) return launch_la<DP, 32, 1, TD>(d, n_seqs, st);   // the wider slice would not fit
+  else {
+  if (ctas64 >= 148) return launch_la<DP, 64, 1, TD>(d, n_seqs, st);
   const long long ctas32 = static_cast<long long>((d.vdim + 31) / 32) * d.heads * n_seqs;
   // a grid that leaves every CTA an SM of its own gets the whole register file (deeper load / FMA overlap); otherwise two per SM
-  return ctas32 <= 148 ? launch_la<DP, 32, 1>(d, n_seqs, st) : launch_la<DP, 32, 2>(d, n_seqs, st);
+  return ctas32 <= 148 ? launch_la<DP, 32, 1, TD>(d, n_seqs, st) : launch_la<DP, 32, 2, TD>(d, n_seqs, st);
+  }
 }
 
 cudaError_t launch_linear_attn_chunked(const RecDev& d, int n_seqs, cudaStream_t st) {
@@ -231,6 +294,14 @@ cudaError_t launch_linear_attn_chunked(const RecDev& d, int n_seqs, cudaStream_t
   if (d.dim <= 32) return launch_la_dp<32>(d, n_seqs, st);
   if (d.dim <= 64) return launch_la_dp<64>(d, n_seqs, st);
   return launch_la_dp<128>(d, n_seqs, st);   // callers keep dim <= 128 here
+}
+
+cudaError_t launch_ssd_chunked(const RecDev& d, int n_seqs, cudaStream_t st) {
+  if (d.dim <= 16) return launch_la_dp<16, true>(d, n_seqs, st);
+  if (d.dim <= 32) return launch_la_dp<32, true>(d, n_seqs, st);
+  if (d.dim <= 64) return launch_la_dp<64, true>(d, n_seqs, st);
+  if (d.dim <= 128) return launch_la_dp<128, true>(d, n_seqs, st);
+  return launch_la_dp<256, true>(d, n_seqs, st);   // callers keep dim <= 256
 }
 
 // ---- tiled windowed attention --------------------------------------------------------------------------------------------
@@ -283,6 +354,7 @@ __global__ void __launch_bounds__(WT_T, BN == 32 ? 2 : 1) window_attn_tiled_kern
       for (int e = 0; e < 4; ++e) acc[r][mm][e] = 0.f;
   const long long kstride = d.k_row, vstride = d.v_row;
   const float sc_mul = head_scale_of(d, h), sc_add = head_bias_of(d, h);
+  const float slope = head_slope_of(d, h), two_over_cap = d.softcap > 0.f ? 2.f / d.softcap : 0.f;
   for (int c0 = 0; c0 < count; c0 += WT_N) {
     __syncthreads();
     if (t < WT_N) {
@@ -321,7 +393,7 @@ __global__ void __launch_bounds__(WT_T, BN == 32 ? 2 : 1) window_attn_tiled_kern
         const int i = ti + 16 * r, j = tj + 16 * c;
         const int p = p_lo + i, kp = kpos_s[j];
         const bool vis = i < rows && kp >= 0 && kp <= p && (d.window <= 0 || p - kp < d.window || kp < d.keep) && (d.chunk <= 0 || kp >= p / d.chunk * d.chunk);
-        const float z = fmaf(sc[r][c], sc_mul, sc_add);
+        const float z = shaped_score(d, fmaf(sc[r][c], sc_mul, sc_add), two_over_cap, slope, p - kp);
         if constexpr (SIG) Ps[i * WT_LDP + j] = vis ? sigmoidf_(z) : 0.f;
         else Ps[i * WT_LDP + j] = vis ? z : -INFINITY;
       }
@@ -447,6 +519,7 @@ __global__ void __launch_bounds__(WH_T) window_attn_heads_kernel(WinDev d, int l
       l[e] = split == 0 ? 1.f : 0.f;
     }
   }
+  const float two_over_cap = d.softcap > 0.f ? 2.f / d.softcap : 0.f;
   const int kj = t & 63, hq = t >> 6;   // score phase: key kj, heads 4 hq .. 4 hq + 3; output phase: channels kj + 64 cc, same heads
   float acc[4][WH_VC];
 #pragma unroll
@@ -482,10 +555,12 @@ __global__ void __launch_bounds__(WH_T) window_attn_heads_kernel(WinDev d, int l
         for (int e = 0; e < 4; ++e) sc[e] = dot4(f4(q0 + e * ldk + c), k4, sc[e]);
       }
       const bool vis = krow_s[kj] >= 0;
+      const int c_key = c0 + kj, dist = pos - (c_key < nA ? c_key : lowB + (c_key - nA));
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int hh = min(h0 + 4 * hq + e, d.heads - 1);   // rows past the group hold no head: never stored
-        Ss[(4 * hq + e) * LDS_ + kj] = vis ? fmaf(sc[e], head_scale_of(d, hh), head_bias_of(d, hh)) : -INFINITY;
+        const float z = fmaf(sc[e], head_scale_of(d, hh), head_bias_of(d, hh));
+        Ss[(4 * hq + e) * LDS_ + kj] = vis ? shaped_score(d, z, two_over_cap, head_slope_of(d, hh), dist) : -INFINITY;
       }
     }
     __syncthreads();

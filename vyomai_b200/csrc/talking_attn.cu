@@ -32,12 +32,6 @@ struct TalkDev {
   void* out; long long ld_out; int out_dt;
 };
 
-// cap * tanh(s / cap) as cap * (1 - 2 / (1 + e^(2 s / cap))): expf and a fast reciprocal, absolute error a few 1e-7 * cap (the softmax
-// that follows depends on score differences, i.e. on absolute error); e^x overflowing to inf gives exactly cap, underflow exactly -cap
-__device__ __forceinline__ float cap_score(float s, float cap, float two_over_cap) {
-  return cap > 0.f ? cap * (1.f - __fdividef(2.f, 1.f + expf(s * two_over_cap))) : s;
-}
-
 // the extra softmax term of head h as (score, present)
 __device__ __forceinline__ bool sink_of(const TalkDev& d, int h, float& s) {
   if (d.sink) { s = ld_as_float(d.sink, d.sink_dt, h); return true; }

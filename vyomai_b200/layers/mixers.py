@@ -1,5 +1,5 @@
 """Sequence mixers and feed-forwards of the packed-step decoder families (models/gelutar.py, models/zugunex.py, models/vazepel.py,
-models/fubinex.py, models/kifetar.py), on the packed-batch kernels of csrc/seqmix.cu, csrc/gated_delta.cu, csrc/latent.cu,
+models/fubinex.py, models/kifetar.py, models/zaparax.py), on the packed-batch kernels of csrc/seqmix.cu, csrc/gated_delta.cu, csrc/ssd.cu, csrc/latent.cu,
 csrc/talking_attn.cu, csrc/parallel_block.cu and csrc/rowwise.cu. Each mixer is built from its config block and its weights, declares what it keeps per sequence
 (`cache_spec`: pages of keys / values, recurrent state slots) and maps the normed layer input h [rows, width] to its
 output; the constants of a mechanism (window, kept tokens, scale, sink, decay, taps, head counts) are constructor
@@ -445,6 +445,88 @@ class HeadDecayDeltaMixer(Mixer):
         return self.o(o)
 
 
+class BiasedAttention(Mixer):
+    """Grouped-query softmax attention without rotation whose scores lose ground with distance: biased q / k / v projections, every head of
+    q and k divided by its root mean square over dim (no weight), q at position p times 1 + q_temp.coef ln(floor((p + 1) / q_temp.every) + 1);
+    score = cap(q . k * scale) - slope_h (i - j), cap(s) = softcap tanh(s / softcap), slope_h = 2^(-8 (h + 1) / heads); a learned sink per
+    head in the denominator. mask = {"size": n}: a query sees the last n positions, its own included. q_temp, softcap, mask, sink and the
+    projection biases each only when the configuration / the weights hold them. Normed keys and values live in pages."""
+
+    def __init__(self, cfg: dict, w: Dict[str, torch.Tensor], eps: float, act_dtype: torch.dtype, tensor_cores: bool,
+                 kv_dtype: torch.dtype = torch.float32):
+        self.heads, self.kv_heads = int(cfg["heads"]), int(cfg["kv_heads"])
+        self.dim, self.vdim = int(cfg["dim"]), int(cfg["vdim"])
+        if self.heads % self.kv_heads:
+            raise ValueError("attention: heads must be a multiple of kv_heads")
+        self.window = int((cfg.get("mask") or {}).get("size", 0))
+        self.scale, self.softcap = float(cfg["scale"]), float(cfg.get("softcap") or 0.0)
+        t = cfg.get("q_temp")
+        self.q_temp = (float(t["coef"]), int(t["every"])) if t else None
+        self.eps, self.act_dtype, self.kv_dtype = eps, act_dtype, kv_dtype
+        dev = w["q"].device
+        self.no_rotation, _ = rotary_frequencies({}, 0, dev)
+        self.slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)], dtype=torch.float64).to(torch.float32).to(dev)
+        self._in = [w["q"], w["k"], w["v"]]
+        self._in_b = [w.get("q.b"), w.get("k.b"), w.get("v.b")]
+        self.sink = w["sink"].contiguous() if "sink" in w else None
+        self.o = Projection(w["o"], tensor_cores)
+
+    def input_weights(self):
+        return self._in
+
+    def input_biases(self):
+        return self._in_b
+
+    def cache_spec(self):
+        return {"pages": (self.kv_heads, self.dim, self.vdim), "states": {}, "kv_dtype": self.kv_dtype}
+
+    def forward(self, parts, batch, cache):
+        q, k, v = parts
+        ops.rope_kv_write(batch, q, k, v, self.no_rotation, cache.k_pool, cache.v_pool, heads=self.heads, kv_heads=self.kv_heads, dim=self.dim,
+                          vdim=self.vdim, rot_dims=0, layout="half", unit_rms=True, eps=self.eps, q_temp=self.q_temp)
+        a = ops.window_attn(batch, q, cache.k_pool, cache.v_pool, heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim,
+                            scale=self.scale, window=self.window, keep_first=0, sink=self.sink, out_dtype=self.act_dtype, softcap=self.softcap,
+                            head_slope=self.slopes)
+        return self.o(a)
+
+
+class StateSpaceMixer(Mixer):
+    """State-space recurrence with one decay per head and token (Mamba-2): W_in h = [z | x | B | C | dt]; x, B and C pass a short causal
+    depthwise convolution with bias and silu; w = softplus(dt + dt_bias), S <- exp(-exp(A_log) w) S + w B x^T (S is state x vdim; B and C
+    shared by heads / groups heads), y = S^T C + D x; y silu(z) is RMS-normed in norm_groups equal runs of columns, times a weight per
+    column, then projected. State and the convolution's last inputs are fp32 per sequence slot (ops.ssd does everything between the two
+    projections)."""
+
+    def __init__(self, cfg: dict, w: Dict[str, torch.Tensor], eps: float, act_dtype: torch.dtype, tensor_cores: bool):
+        self.heads, self.groups = int(cfg["heads"]), int(cfg["groups"])
+        self.dim, self.vdim, self.taps, self.norm_groups = int(cfg["state"]), int(cfg["vdim"]), int(cfg["conv"]), int(cfg["norm_groups"])
+        inner, gn = self.heads * self.vdim, self.groups * self.dim
+        if self.heads % self.groups or inner % self.norm_groups:
+            raise ValueError("state space: groups must divide heads and norm_groups the heads' columns")
+        self.channels = inner + 2 * gn
+        self.eps, self.act_dtype = eps, act_dtype
+        cuts = [inner, inner, gn, gn, self.heads]
+        self._in = list(torch.split(w["in"], cuts, 0))   # z | x | B | C | dt
+        self.conv_w, self.conv_b = w["conv"].contiguous(), w["conv.b"].contiguous() if "conv.b" in w else None
+        self.dt_bias, self.a_log, self.skip = w["dt_bias"].contiguous(), w["A_log"].contiguous(), w["D"].contiguous()
+        self.norm = w["norm"].contiguous()
+        self.o = Projection(w["o"], tensor_cores)
+
+    def input_weights(self):
+        return self._in
+
+    def cache_spec(self):
+        return {"pages": None, "states": {"S": (self.heads, self.dim, self.vdim), "conv": (self.taps, self.channels), "done": (1,)},
+                "state_dtypes": {"done": torch.int32}}
+
+    def forward(self, parts, batch, cache):
+        z, x, b, c, dt = parts
+        y = ops.ssd(batch, x, b, c, dt, z, self.conv_w, self.conv_b, cache.states["conv"], self.dt_bias, self.a_log, self.skip, self.norm,
+                    cache.states["S"], cache.states["done"], heads=self.heads, groups=self.groups, dim=self.dim, vdim=self.vdim, taps=self.taps,
+                    norm_groups=self.norm_groups, norm_eps=self.eps, out_dtype=self.act_dtype)
+        return self.o(y)
+
+
 class LatentAttention(Mixer):
     """Attention whose keys and values are linear images of a cached low-rank latent: per token the cache holds the RMS-normed
     latent c [rank] and one rotated key part kr [rot_dim] shared by the heads. Head h scores (qn_h . W_uk_h c + qr_h . kr) * scale
@@ -678,9 +760,11 @@ class MoEFeedForward:
 
     Router (`router`): "sigmoid" scores or the "softmax" over all experts; with `groups` = (count, keep) only members of the `keep`
     best of `count` runs of neighbouring experts are eligible; the `top` largest eligible scores are kept and, with `normalize`,
-    divided by their sum; times `route_scale`.
+    divided by their sum; times `route_scale`. When the weights hold `correction`, the choice is by score + correction. The last `identity`
+    router outputs are identity experts: no weights, their output is h (see `forward_parts`).
     Expert (`form`): "plain" = W_down act(W_up h); "glu" = W_down (g sigmoid(alpha g) (u + 1)) with g = min(W_gate h, limit),
-    u = clamp(W_up h, +-limit) (the shared expert with `shared_limit`). The shared expert is weighted by sigmoid(w_sg . h) when the
+    u = clamp(W_up h, +-limit) (the shared expert with `shared_limit`); "swiglu" = W_down (silu(W_gate h) * W_up h), gate and up rows
+    interleaved so that the product's epilogue can do it. The shared expert is weighted by sigmoid(w_sg . h) when the
     weights hold `shared.sg`, by 1 otherwise.
 
     Two exact forms of the same sum. Single tokens and short steps (also every CUDA-graph-captured step: no host decision)
@@ -698,19 +782,26 @@ class MoEFeedForward:
     def __init__(self, w: Dict[str, torch.Tensor], experts: int, top: int, route_scale: float, act_dtype: torch.dtype, tensor_cores: bool,
                  act: str = "relu2", shared: bool = False, sorted_min_rows: int = 128, force_sorted: bool = False, router: str = "sigmoid",
                  groups: Optional[Tuple[int, int]] = None, normalize: bool = True, form: str = "plain", limit: float = 0.0,
-                 shared_limit: float = 0.0, alpha: float = 1.702, router_logits: bool = True):
+                 shared_limit: float = 0.0, alpha: float = 1.702, router_logits: bool = True, identity: int = 0):
         self.experts, self.top, self.route_scale = int(experts), int(top), float(route_scale)
         self.act_dtype, self.act, self.sorted_min_rows, self.force_sorted = act_dtype, act, int(sorted_min_rows), bool(force_sorted)
         self.router_kind, self.normalize = router, bool(normalize)
         self.groups, self.keep_groups = (int(groups[0]), int(groups[1])) if groups and int(groups[0]) > 1 else (0, 0)
         if self.groups and (self.experts % self.groups or not 0 < self.keep_groups <= self.groups or self.top > self.keep_groups * (self.experts // self.groups)):
             raise ValueError("experts: the groups must divide the experts, and the kept groups hold at least `top` experts")
-        if form not in ("plain", "glu"):
+        if form not in ("plain", "glu", "swiglu"):
             raise ValueError(f"experts: unknown form {form!r}")
-        self.glu, self.limit, self.shared_limit, self.alpha = form == "glu", float(limit), float(shared_limit), float(alpha)
+        self.swiglu = form == "swiglu"
+        self.glu, self.limit, self.shared_limit, self.alpha = form != "plain", float(limit), float(shared_limit), float(alpha)
+        self.identity = int(identity)
+        if self.identity and self.groups:
+            raise ValueError("experts: identity experts and groups are not combined")
+        self.correction = w["correction"].contiguous() if "correction" in w else None
         E = self.experts
         self.ff = w["e0.up"].shape[0]
-        hid = (lambda pre: torch.cat([w[pre + "gate"], w[pre + "up"]], 0)) if self.glu else (lambda pre: w[pre + "up"])
+        from .gated import interleave_gate_up
+        hid = (lambda pre: interleave_gate_up(w[pre + "gate"], w[pre + "up"])) if self.swiglu else \
+            (lambda pre: torch.cat([w[pre + "gate"], w[pre + "up"]], 0)) if self.glu else (lambda pre: w[pre + "up"])
         ups = [hid(f"e{e}.") for e in range(E)]
         downs = [w[f"e{e}.down"] for e in range(E)]
         self.shared_ff = 0
@@ -744,6 +835,13 @@ class MoEFeedForward:
 
     def _hidden(self, proj: Projection, x: torch.Tensor, dense: Optional[torch.Tensor], experts: int, shared_ff: int, sg, wide: bool) -> torch.Tensor:
         """The activated (and, with `dense`, weighted) hidden rows of `experts` experts and / or the shared expert, in the activation dtype."""
+        if self.swiglu:
+            if wide and proj.fuses_swiglu(x, self.act_dtype):   # prompt-sized: the activation in the product's epilogue, weighted in place
+                u = proj(x, act="swiglu", out_dtype=self.act_dtype)
+                return u if dense is None and sg is None else ops.moe_scale(u, dense, experts=experts, ff=self.ff if experts else 1, shared_ff=shared_ff,
+                                                                             shared_gate=sg, out_dtype=self.act_dtype, out=u)
+            return ops.moe_glu(proj(x), dense, experts=experts, ff=self.ff, shared_ff=shared_ff, limit=0.0, alpha=1.0, out_dtype=self.act_dtype,
+                               interleaved=True, shift=False, shared_gate=sg if shared_ff else None)
         if self.glu:
             u = proj(x)   # fp32 pre-activations: the clamps and the gate see the accumulator, rounded once after the activation
             return ops.moe_glu(u, dense, experts=experts, ff=self.ff, shared_ff=shared_ff, limit=self.limit, shared_limit=self.shared_limit,
@@ -757,21 +855,30 @@ class MoEFeedForward:
     def forward(self, h: torch.Tensor, batch, logits: Optional[torch.Tensor] = None) -> torch.Tensor:
         """h: the layer input in the activation dtype; logits: the router's fp32 logits (and the shared gate's) when the caller has them
         already. Returns fp32 [rows, width]."""
+        if self.identity:
+            raise _lib.VyomError("experts: a layer with identity experts takes forward_parts")
+        return self.forward_parts(h, batch, logits)[0]
+
+    def forward_parts(self, h: torch.Tensor, batch, logits: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+        """(y fp32 [rows, width], weight fp32 [rows] or None): the layer's output is y + weight * h, the second term being the chosen identity
+        experts' (the caller adds it where it reads y, without a pass of its own)."""
         E, rows = self.experts, h.shape[0]
         z = logits if logits is not None else self.router(h)
+        scored = E + self.identity
         sorted_form = batch.max_new > 1 and rows >= self.sorted_min_rows and (self.force_sorted or self._sorted_is_faster(rows))
-        idx, wt, dense = ops.moe_route(z, E, self.top, self.route_scale, dense=not sorted_form, kind=self.router_kind, groups=self.groups,
-                                       keep_groups=self.keep_groups, normalize=self.normalize)
-        sg = z[:, E:E + 1] if self.shared_gated else None
+        idx, wt, dense, *rest = ops.moe_route(z, scored, self.top, self.route_scale, dense=not sorted_form, kind=self.router_kind, groups=self.groups,
+                                              keep_groups=self.keep_groups, normalize=self.normalize, correction=self.correction, identity=self.identity)
+        ident = rest[0] if rest else None
+        sg = z[:, scored:scored + 1] if self.shared_gated else None
         if not sorted_form:
             # few rows: fp32 hidden activations, weighted, rounded once. Prompt-sized steps write them in the activation dtype from
             # the product's epilogue and weight them in place (half the bytes of the step's largest tensor, one more rounding)
             wide = rows > 32 and self.act_dtype != torch.float32
-            return self.down_all(self._hidden(self.up_all, h, dense, E, self.shared_ff, sg, wide))
-        counts, offsets, perm, inv = ops.moe_sort(idx, E)
+            return self.down_all(self._hidden(self.up_all, h, dense, E, self.shared_ff, sg, wide)), ident
+        counts, offsets, perm, inv = ops.moe_sort(idx, scored)
         xg = ops.moe_gather(h, perm, self.top, self.act_dtype)
         off = offsets.cpu().tolist()   # the one host decision of a prompt step: how many rows each expert got
-        part = torch.empty((rows * self.top, self.down_all.out_features), device=h.device, dtype=torch.float32)
+        part = torch.empty((max(off[E], 1), self.down_all.out_features), device=h.device, dtype=torch.float32)
         for e in range(E):
             a, b = off[e], off[e + 1]
             if b > a:
@@ -779,4 +886,4 @@ class MoEFeedForward:
         ys = None
         if self.shared_ff:
             ys = self.down_s(self._hidden(self.up_s, h, None, 0, self.shared_ff, sg, False))
-        return ops.moe_combine(part, inv, wt, addend=ys)
+        return ops.moe_combine(part, inv, wt, addend=ys, idx=idx if self.identity else None, routed=E), ident

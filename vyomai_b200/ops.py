@@ -986,14 +986,29 @@ def poly_norm(x: torch.Tensor, coef, *, eps: float, out_dtype: Optional[torch.dt
     return out
 
 
+CLOSE_KIND = {"layer": C["VY_CLOSE_LAYER"], "rms": C["VY_CLOSE_RMS"], "rms_centred": C["VY_CLOSE_RMS_CENTRED"]}
+
+
 def sandwich_norm(x: torch.Tensor, y: Optional[torch.Tensor] = None, norm1=None, norm2=None, *, eps: float, x_out: Optional[torch.Tensor] = None,
-                  copy_out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, row_index: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
-    """One pass over packed fp32 rows: s = x + LayerNorm1(y) (y None: s = x), written to x_out (fp32, may be x) and copy_out (its own
-    dtype) when given; returns LayerNorm2(s) in out_dtype (norm2 None: nothing). norm1 / norm2: (weight, bias) pairs, all one dtype."""
+                  copy_out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, row_index: Optional[torch.Tensor] = None,
+                  kind: str = "layer", second: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> Optional[torch.Tensor]:
+    """One pass over packed fp32 rows: s = x + N1(y) (y None: s = x), written to x_out (fp32, may be x) and copy_out (its own dtype) when
+    given; returns N2(s) in out_dtype (norm2 None: nothing). kind: what norms are, "layer" (layer norm; norm1 / norm2 are (weight, bias)
+    pairs), "rms" or "rms_centred" (RMS norm times w or 1 + w; norm1 / norm2 are the weights); all one dtype. second = (u [rows, width],
+    coef fp32 [rows]): y + coef * u is normed in y's place."""
+    if kind not in CLOSE_KIND:
+        raise _lib.VyomError(f"sandwich_norm: unknown kind {kind!r}")
+    if kind != "layer":
+        norm1, norm2 = (norm1, None) if norm1 is not None else None, (norm2, None) if norm2 is not None else None
     w1, b1 = norm1 if norm1 is not None else (None, None)
     w2, b2 = norm2 if norm2 is not None else (None, None)
     ws = [t for t in (w1, b1, w2, b2) if t is not None]
-    _need_cuda(x, y, x_out, copy_out, row_index, *ws)
+    u, u_coef = second if second is not None else (None, None)
+    _need_cuda(x, y, x_out, copy_out, row_index, u, u_coef, *ws)
+    if u is not None:
+        _rows2d(u, "sandwich_norm second")
+        if y is None or u.shape != x.shape or u_coef.dtype != torch.float32 or u_coef.numel() != x.shape[0] or not u_coef.is_contiguous():
+            raise _lib.VyomError("sandwich_norm: the second result has x's shape and one fp32 weight per row, beside y")
     for t, n in ((x, "x"), (y, "y"), (x_out, "x_out"), (copy_out, "copy_out")):
         if t is not None:
             _rows2d(t, f"sandwich_norm {n}")
@@ -1007,7 +1022,8 @@ def sandwich_norm(x: torch.Tensor, y: Optional[torch.Tensor] = None, norm1=None,
     _lib.call("vy_sandwich_norm", "VySandwichNorm", rows=rows, width=x.shape[1], row_index=_ptr(row_index), x=x.data_ptr(), ldx=x.stride(0), y=_ptr(y),
               ldy=y.stride(0) if y is not None else 0, w1=_ptr(w1), b1=_ptr(b1), w2=_ptr(w2), b2=_ptr(b2), w_dtype=_dt(ws[0]) if ws else 0, eps=float(eps),
               copy_dtype=_dt(copy_out) if copy_out is not None else 0, out_dtype=_dt(out) if out is not None else 0, stream=_stream(),
-              **opt(x_out, "x_out"), **opt(copy_out, "copy"), **opt(out, "out"))
+              norm_kind=CLOSE_KIND[kind], u_dtype=_dt(u) if u is not None else 0, u_coef=_ptr(u_coef),
+              **opt(x_out, "x_out"), **opt(copy_out, "copy"), **opt(out, "out"), **opt(u, "u"))
     return out
 
 
@@ -1043,6 +1059,26 @@ def embed_rows(ids: torch.Tensor, table: torch.Tensor, scale: float, out_dtype: 
     return out
 
 
+def pair_embed(batch: PackedBatch, ids: torch.Tensor, table: torch.Tensor, scale: float, pairs: torch.Tensor, prev_state: torch.Tensor, *, mul_prev: int,
+               mul_cur: int, out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
+    """scale * table[id] + pairs[(previous id * mul_prev + id * mul_cur) mod buckets], buckets = len(pairs) - 1; position 0 reads the last
+    row of `pairs`. prev_state [slots, ..] int32 carries each sequence's last id between steps and is advanced."""
+    _need_cuda(ids, table, pairs, prev_state)
+    _rows2d(table, "pair_embed table")
+    _rows2d(pairs, "pair_embed pairs")
+    if ids.dtype != torch.int32 or prev_state.dtype != torch.int32 or not prev_state.is_contiguous() or prev_state[0].numel() != 1:
+        raise _lib.VyomError("pair_embed: ids and prev_state (one per slot) are int32")
+    if table.dtype != pairs.dtype or table.shape[1] != pairs.shape[1]:
+        raise _lib.VyomError("pair_embed: the two tables share dtype and width")
+    out = torch.empty((ids.numel(), table.shape[1]), device=table.device, dtype=out_dtype)
+    buckets = pairs.shape[0] - 1
+    _lib.call("vy_pair_embed", "VyPairEmbed", ids=ids.data_ptr(), width=table.shape[1], vocab=table.shape[0], table=table.data_ptr(), ld_table=table.stride(0),
+              pairs=pairs.data_ptr(), ld_pairs=pairs.stride(0), table_dtype=_dt(table), scale=float(scale), mul_prev=int(mul_prev) % buckets,
+              mul_cur=int(mul_cur) % buckets, buckets=buckets, prev_state=prev_state.data_ptr(), out=out.data_ptr(), ld_out=out.stride(0), out_dtype=_dt(out),
+              stream=_stream(), **batch._kw())
+    return out
+
+
 def kv_page_write(batch: PackedBatch, k: torch.Tensor, v: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor) -> None:
     _need_cuda(k, v, k_pool, v_pool)
     _rows2d(k, "kv_page_write k")
@@ -1060,18 +1096,20 @@ ATTN_WEIGHTS = {"softmax": C["VY_ATTN_SOFTMAX"], "sigmoid": C["VY_ATTN_SIGMOID"]
 def window_attn(batch: PackedBatch, q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, *, heads: int, kv_heads: int, dim: int,
                 vdim: int, scale: float, window: int, keep_first: int, sink: Optional[torch.Tensor] = None,
                 gate: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, k_row: int = 0, v_row: int = 0, chunk: int = 0, out_scale: float = 1.0,
-                weights: str = "softmax", head_scale: Optional[torch.Tensor] = None, head_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                weights: str = "softmax", head_scale: Optional[torch.Tensor] = None, head_bias: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                head_slope: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of the step's queries over the paged pools (which already hold the step's keys): causal, restricted to the last
     `window` positions plus the first `keep_first` ones (or, with `chunk`, to the query's own block of `chunk` consecutive positions
     counted from position 0), optional per-head sink in the softmax denominator, optional per-head
     sigmoid output gate. weights: "softmax", or "sigmoid" (the weight of a visible key is sigmoid(score), not normalised over keys);
-    head_scale / head_bias: fp32 [heads], score = q.k * scale * head_scale[h] + head_bias[h]. k_row / v_row: row strides of the pools in elements when they are not kv_heads * dim | vdim (two views of
+    head_scale / head_bias: fp32 [heads], score = q.k * scale * head_scale[h] + head_bias[h]; then softcap > 0: cap tanh(score / cap); head_slope (fp32
+    [heads]): minus head_slope[h] times the distance between query and key. k_row / v_row: row strides of the pools in elements when they are not kv_heads * dim | vdim (two views of
     one pool)."""
-    _need_cuda(q, k_pool, v_pool, sink, gate, head_scale, head_bias)
+    _need_cuda(q, k_pool, v_pool, sink, gate, head_scale, head_bias, head_slope)
     _rows2d(q, "window_attn q")
-    for t in (head_scale, head_bias):
+    for t in (head_scale, head_bias, head_slope):
         if t is not None and (t.dtype != torch.float32 or t.numel() != heads or not t.is_contiguous()):
-            raise _lib.VyomError("window_attn: head_scale / head_bias are contiguous fp32 [heads]")
+            raise _lib.VyomError("window_attn: head_scale / head_bias / head_slope are contiguous fp32 [heads]")
     out = torch.empty((q.shape[0], heads * vdim), device=q.device, dtype=out_dtype or q.dtype)
     ws = None
     if batch.max_new == 1 and heads // kv_heads >= 8:   # the heads-as-rows form splits keys over CTAs and merges from a scratch buffer
@@ -1082,7 +1120,8 @@ def window_attn(batch: PackedBatch, q: torch.Tensor, k_pool: torch.Tensor, v_poo
               window=int(window), keep_first=int(keep_first), sink=_ptr(sink), sink_dtype=_dt(sink) if sink is not None else 0,
               gate=_ptr(gate), ld_gate=gate.stride(0) if gate is not None else 0, gate_dtype=_dt(gate) if gate is not None else 0,
               out=out.data_ptr(), ld_out=out.stride(0), out_dtype=_dt(out), k_row=int(k_row), v_row=int(v_row), stream=_stream(), chunk=int(chunk), out_scale=float(out_scale),
-              weight_kind=ATTN_WEIGHTS[weights], head_scale=_ptr(head_scale), head_bias=_ptr(head_bias), **batch._kw(pages=True, slots=False))
+              weight_kind=ATTN_WEIGHTS[weights], head_scale=_ptr(head_scale), head_bias=_ptr(head_bias), softcap=float(softcap), head_slope=_ptr(head_slope),
+              **batch._kw(pages=True, slots=False))
     return out
 
 
@@ -1120,30 +1159,38 @@ ROUTE_KIND = {"sigmoid": C["VY_ROUTE_SIGMOID"], "softmax": C["VY_ROUTE_SOFTMAX"]
 
 
 def moe_route(logits: torch.Tensor, experts: int, top: int, scale: float, dense: bool = True, kind: str = "sigmoid", groups: int = 0,
-              keep_groups: int = 0, normalize: bool = True):
+              keep_groups: int = 0, normalize: bool = True, correction: Optional[torch.Tensor] = None, identity: int = 0):
     """fp32 logits [rows, >= experts] -> (idx [rows, top] int32, weight [rows, top] fp32, dense [rows, experts] fp32 or None). kind: the
     scores are sigmoids or the softmax over all experts; groups > 1: only members of the keep_groups best runs of neighbours are
-    eligible; normalize: the chosen scores are divided by their sum (else they are the weights as they are)."""
-    _need_cuda(logits)
+    eligible; normalize: the chosen scores are divided by their sum (else they are the weights as they are). correction [experts]: added to
+    the scores for the choice only. With identity > 0 the last `identity` of the experts have no weights: dense covers the others, and a
+    fourth result, fp32 [rows], is the summed weight of each row's chosen identity experts."""
+    _need_cuda(logits, correction)
+    if correction is not None and (correction.numel() != experts or not correction.is_contiguous()):
+        raise _lib.VyomError("moe_route: correction is contiguous [experts]")
     _rows2d(logits, "moe_route logits")
     if logits.dtype != torch.float32:
         raise _lib.VyomError("moe_route: logits are fp32")
     rows = logits.shape[0]
     idx = torch.empty((rows, top), device=logits.device, dtype=torch.int32)
     wt = torch.empty((rows, top), device=logits.device, dtype=torch.float32)
-    dn = torch.empty((rows, experts), device=logits.device, dtype=torch.float32) if dense else None
+    dn = torch.empty((rows, experts - identity), device=logits.device, dtype=torch.float32) if dense else None
+    ident = torch.empty(rows, device=logits.device, dtype=torch.float32) if identity > 0 else None
     _lib.call("vy_moe_route", "VyMoeRoute", rows=rows, experts=experts, top=top, logits=logits.data_ptr(), ld_logits=logits.stride(0),
               scale=float(scale), idx=idx.data_ptr(), weight=wt.data_ptr(), dense=_ptr(dn), stream=_stream(), kind=ROUTE_KIND[kind],
-              groups=int(groups), keep_groups=int(keep_groups), raw_weights=0 if normalize else 1)
-    return idx, wt, dn
+              groups=int(groups), keep_groups=int(keep_groups), raw_weights=0 if normalize else 1, correction=_ptr(correction),
+              correction_dtype=_dt(correction) if correction is not None else 0, identity=int(identity), ident=_ptr(ident))
+    return (idx, wt, dn) if ident is None else (idx, wt, dn, ident)
 
 
 def moe_glu(h: torch.Tensor, dense: Optional[torch.Tensor], *, experts: int, ff: int, shared_ff: int, limit: float, shared_limit: float = 0.0,
-            alpha: float = 1.702, out_dtype: torch.dtype, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+            alpha: float = 1.702, out_dtype: torch.dtype, out: Optional[torch.Tensor] = None, interleaved: bool = False, shift: bool = True,
+            shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Gated experts' activation over h [rows, experts * 2 ff + 2 shared_ff] (per expert [gate | up]): min(gate, limit) *
     sigmoid(alpha * .) * (clamp(up, +-limit) + 1), times the routing weight dense[row, e] (None = 1); the shared block last, with its own
-    limit and weight 1. Returns [rows, experts * ff + shared_ff]."""
-    _need_cuda(h, dense, out)
+    limit and weight 1, or sigmoid(shared_gate[row, 0]). interleaved: gate and up columns alternate; shift=False: times the up half itself,
+    not it + 1 (with alpha 1 and no limit: silu(gate) * up). Returns [rows, experts * ff + shared_ff]."""
+    _need_cuda(h, dense, out, shared_gate)
     _rows2d(h, "moe_glu h")
     if h.shape[1] != 2 * (experts * ff + shared_ff):
         raise _lib.VyomError(f"moe_glu: {h.shape[1]} columns, expected {2 * (experts * ff + shared_ff)}")
@@ -1151,7 +1198,8 @@ def moe_glu(h: torch.Tensor, dense: Optional[torch.Tensor], *, experts: int, ff:
         out = torch.empty((h.shape[0], _round_up(experts * ff + shared_ff, 8)), device=h.device, dtype=out_dtype)[:, :experts * ff + shared_ff]
     _lib.call("vy_moe_glu", "VyMoeGlu", rows=h.shape[0], experts=experts, ff=ff, shared_ff=shared_ff, h=h.data_ptr(), ldh=h.stride(0), h_dtype=_dt(h),
               dense=_ptr(dense), ld_dense=dense.stride(0) if dense is not None else 0, limit=float(limit), shared_limit=float(shared_limit),
-              alpha=float(alpha), out=out.data_ptr(), ld_out=out.stride(0), out_dtype=_dt(out), stream=_stream())
+              alpha=float(alpha), out=out.data_ptr(), ld_out=out.stride(0), out_dtype=_dt(out), stream=_stream(), interleaved=1 if interleaved else 0,
+              no_shift=0 if shift else 1, shared_gate=_ptr(shared_gate), ld_gate=shared_gate.stride(0) if shared_gate is not None else 0)
     return out
 
 
@@ -1210,11 +1258,13 @@ def depth_mix(x: torch.Tensor, y1: torch.Tensor, g1: Optional[torch.Tensor], y2:
 def rope_kv_write(batch: PackedBatch, q: Optional[torch.Tensor], k: Optional[torch.Tensor], v: Optional[torch.Tensor], inv_freq: torch.Tensor,
                   k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor], *, heads: int, kv_heads: int, dim: int, vdim: int, rot_dims: int,
                   layout: str = "pairs", rot_scale: float = 1.0, unit_rms: bool = False, eps: float = 0.0, q_scale: float = 1.0, k_scale: float = 1.0,
-                  k_out: Optional[torch.Tensor] = None, q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None) -> None:
+                  k_out: Optional[torch.Tensor] = None, q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None,
+                  q_temp: Optional[Tuple[float, int]] = None) -> None:
     """Rotates q in place by position, rotates k into k_pool and copies v into v_pool at each token's page row (one launch).
     layout: "pairs" turns entries (2i, 2i + 1), "half" entries (i, i + rot_dims / 2); rot_scale multiplies cos and sin; unit_rms divides
     every rotated head of q and k by sqrt(mean of its squares + eps); q_norm / k_norm (weights [dim], shared by the heads) RMS-norm every
-    head of q / k BEFORE the rotation instead; q_scale / k_scale multiply the heads last. v may be k itself (the values are the keys as
+    head of q / k BEFORE the rotation instead; q_scale / k_scale multiply the heads last; q_temp = (coef, every) also multiplies the query at
+    position p by 1 + coef ln(floor((p + 1) / every) + 1). v may be k itself (the values are the keys as
     projected). Without pools the rotated keys go to k_out [rows, kv_heads * dim] (may be k itself; v is not touched)."""
     _need_cuda(q, k, v, inv_freq, k_pool, v_pool, k_out, q_norm, k_norm)
     nw = q_norm if q_norm is not None else k_norm
@@ -1241,6 +1291,7 @@ def rope_kv_write(batch: PackedBatch, q: Optional[torch.Tensor], k: Optional[tor
               half_layout=1 if layout == "half" else 0, unit_rms=1 if unit_rms else 0, eps=float(eps), rot_scale=float(rot_scale), q_scale=float(q_scale),
               k_scale=float(k_scale), k_out=_ptr(k_out), ld_k_out=k_out.stride(0) if k_out is not None else 0,
               q_norm=_ptr(q_norm), k_norm=_ptr(k_norm), norm_dtype=_dt(nw) if nw is not None else 0,
+              q_temp=float(q_temp[0]) if q_temp is not None else 0.0, q_temp_every=int(q_temp[1]) if q_temp is not None else 0,
               **batch._kw(pages=paged, slots=False))
 
 
@@ -1312,16 +1363,18 @@ def moe_gather(x: torch.Tensor, perm: torch.Tensor, top: int, out_dtype: torch.d
     return out
 
 
-def moe_combine(part: torch.Tensor, inv: torch.Tensor, weight: torch.Tensor, addend: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[row] = addend[row] + sum_k weight[row, k] * part[inv[row * top + k]] (fp32)."""
-    _need_cuda(part, inv, weight, addend)
+def moe_combine(part: torch.Tensor, inv: torch.Tensor, weight: torch.Tensor, addend: Optional[torch.Tensor] = None, idx: Optional[torch.Tensor] = None,
+                routed: int = 0) -> torch.Tensor:
+    """out[row] = addend[row] + sum_k weight[row, k] * part[inv[row * top + k]] (fp32); with idx [rows, top] the pairs whose expert is
+    >= routed have no row in `part` and are left out."""
+    _need_cuda(part, inv, weight, addend, idx)
     _rows2d(part, "moe_combine part")
     rows, top = weight.shape
     out = torch.empty((rows, part.shape[1]), device=part.device, dtype=torch.float32)
     _lib.call("vy_moe_combine", "VyMoeCombine", rows=rows, top=top, width=part.shape[1], inv=inv.data_ptr(), weight=weight.data_ptr(),
               part=part.data_ptr(), ld_part=part.stride(0), part_dtype=_dt(part), addend=_ptr(addend),
               ld_addend=addend.stride(0) if addend is not None else 0, addend_dtype=_dt(addend) if addend is not None else 0,
-              out=out.data_ptr(), ld_out=out.stride(0), out_dtype=_dt(out), stream=_stream())
+              out=out.data_ptr(), ld_out=out.stride(0), out_dtype=_dt(out), stream=_stream(), idx=_ptr(idx), routed=int(routed))
     return out
 
 
@@ -1429,4 +1482,41 @@ def gated_delta(batch: PackedBatch, q: torch.Tensor, k: torch.Tensor, v: torch.T
               conv_state=conv_state.data_ptr(), a_log=a_log.data_ptr(), norm=norm.data_ptr(), w_dtype=_dt(norm), heads=heads, kv_heads=kv_heads, dim=dim,
               vdim=vdim, unit_eps=float(unit_eps), norm_eps=float(norm_eps), state=state.data_ptr(), out=out.data_ptr(), ld_out=out.stride(0),
               out_dtype=_dt(out), workspace=_ptr(ws), workspace_floats=need, stream=_stream(), **batch._kw())
+    return out
+
+
+def ssd(batch: PackedBatch, x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, dt: torch.Tensor, gate: Optional[torch.Tensor], conv_w: torch.Tensor,
+        conv_b: Optional[torch.Tensor], conv_state: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor, norm: torch.Tensor,
+        state: torch.Tensor, tickets: torch.Tensor, *, heads: int, groups: int, dim: int, vdim: int, taps: int, norm_groups: int, norm_eps: float,
+        gate_act: Optional[str] = "silu", out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """State-space recurrence with one decay per head and token, from the raw fp32 projections x / gate [rows, heads * vdim], b / c
+    [rows, groups * dim] and dt [rows, heads] to the gated, normed read-out [rows, heads * vdim]: causal convolution (conv_w [channels of
+    x | b | c, taps], last column = current token, bias conv_b; ring conv_state [slots, taps, channels]) and silu, step w = softplus(dt +
+    dt_bias), S <- exp(-exp(a_log) w) S + w b x^T, y = S^T c + skip x, times gate_act(gate), RMS norm of `norm_groups` equal runs of columns,
+    times norm [heads * vdim]. tickets [slots, ..]: int32 zeros, scratch of the single-token form."""
+    _need_cuda(x, b, c, dt, gate, conv_w, conv_b, conv_state, dt_bias, a_log, skip, norm, state, tickets)
+    inner, gn = heads * vdim, groups * dim
+    for t, n, w in ((x, "x", inner), (b, "b", gn), (c, "c", gn), (dt, "dt", heads), (gate, "gate", inner)):
+        if t is not None:
+            _rows2d(t, f"ssd {n}")
+            if t.dtype != torch.float32 or t.shape[1] < w:
+                raise _lib.VyomError(f"ssd: {n} is fp32 and as wide as its heads")
+    ws_ = [(conv_w, (inner + 2 * gn, taps)), (conv_b, (inner + 2 * gn,)), (dt_bias, (heads,)), (a_log, (heads,)), (skip, (heads,)), (norm, (inner,))]
+    if any(t is not None and (tuple(t.shape) != shp or not t.is_contiguous() or t.dtype != norm.dtype) for t, shp in ws_):
+        raise _lib.VyomError("ssd: conv_w [channels, taps], conv_b [channels], dt_bias / a_log / skip [heads], norm [heads * vdim] are contiguous and share a dtype")
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (heads, dim, vdim) or conv_state.dtype != torch.float32 or \
+            not conv_state.is_contiguous() or tuple(conv_state.shape[1:]) != (taps, inner + 2 * gn):
+        raise _lib.VyomError("ssd: state [slots, heads, dim, vdim] and conv_state [slots, taps, channels] are contiguous fp32")
+    if tickets.dtype != torch.int32 or not tickets.is_contiguous() or tickets.numel() != state.shape[0]:
+        raise _lib.VyomError("ssd: tickets are int32, one per slot")
+    rows = x.shape[0]
+    out = torch.empty((rows, _round_up(inner, 8)), device=x.device, dtype=out_dtype or torch.float32)[:, :inner]
+    need = int(_lib.lib().vy_ssd_workspace_floats(rows, batch.n_seqs, batch.max_new, heads, groups, dim, vdim))
+    ws = torch.empty(need, device=x.device, dtype=torch.float32)
+    _lib.call("vy_ssd", "VySsd", rows=rows, x=x.data_ptr(), ldx=x.stride(0), b=b.data_ptr(), ldb=b.stride(0), c=c.data_ptr(), ldc=c.stride(0), dt=dt.data_ptr(),
+              ld_dt=dt.stride(0), gate=_ptr(gate), ld_gate=gate.stride(0) if gate is not None else 0, gate_act=UACT[gate_act], conv_w=conv_w.data_ptr(),
+              conv_b=_ptr(conv_b), taps=taps, conv_state=conv_state.data_ptr(), dt_bias=dt_bias.data_ptr(), a_log=a_log.data_ptr(), skip=skip.data_ptr(),
+              norm=norm.data_ptr(), w_dtype=_dt(norm), heads=heads, groups=groups, dim=dim, vdim=vdim, norm_groups=norm_groups, norm_eps=float(norm_eps),
+              state=state.data_ptr(), tickets=tickets.data_ptr(), out=out.data_ptr(), ld_out=out.stride(0), out_dtype=_dt(out), workspace=ws.data_ptr(),
+              workspace_floats=need, stream=_stream(), **batch._kw())
     return out

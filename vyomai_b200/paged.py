@@ -226,7 +226,8 @@ class HybridCacheManager:
     [num_blocks, block_size, kv_heads, dim | vdim] addressed through each sequence's block list — the same page scheme as
     PagedKVManager above (vdim 0: one pool only, for mixers whose values are part of the key row); a mixer that declares
     "pages_from": (layer, mixer) owns no pool and is handed the view of the mixer it names (layers that attend over another
-    layer's cached rows); recurrent mixers get fp32 tensors [num_slots, *shape] addressed by the sequence's slot. Both
+    layer's cached rows); recurrent mixers get tensors [num_slots, *shape] addressed by the sequence's slot (fp32 unless
+    "state_dtypes" names another type for a state). Both
     grow on demand, so `max_tokens` / `max_seqs` are sizing hints, not limits. A slot or page handed out again is not
     cleared: a sequence whose first position is 0 never reads what its slot held, and pages are written before they are
     read."""
@@ -280,7 +281,7 @@ class HybridCacheManager:
         for layer, views in zip(self._specs, self.views):
             for spec, view in zip(layer, views):
                 for name, shape in spec["states"].items():
-                    new = torch.zeros((new_total,) + tuple(shape), device=self.device, dtype=torch.float32)
+                    new = torch.zeros((new_total,) + tuple(shape), device=self.device, dtype=spec.get("state_dtypes", {}).get(name, torch.float32))
                     if name in view.states:
                         new[: self.num_slots] = view.states[name]
                     view.states[name] = new

@@ -52,6 +52,11 @@ def _kifetar(path, **kw):
     return KifetarForCausalLM.from_pretrained(path, **kw)
 
 
+def _zaparax(path, **kw):
+    from .models.zaparax import ZaparaxForCausalLM
+    return ZaparaxForCausalLM.from_pretrained(path, **kw)
+
+
 def _custom_lm(path, dtype=torch.bfloat16, device=None, **kw):
     """The RMSNorm / SwiGLU / RoPE decoder (models/custom_transformer.py): config.json holds its Config fields, the checkpoint
     its state_dict."""
@@ -70,4 +75,5 @@ register_model("Zugunex", _zugunex)
 register_model("Vazepel", _vazepel)
 register_model("Fubinex", _fubinex)
 register_model("Kifetar", _kifetar)
+register_model("Zaparax", _zaparax)
 register_model("ModelForCausalLM", _custom_lm)
