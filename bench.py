@@ -1654,6 +1654,155 @@ def run_kifetar(args):
                       "clocks": sampler.result(), "l2": "160 MB buffer rewritten between timed prefill iterations"}))
 
 
+# ------------------------------------------------------------------------------------------------
+# --workload zaparax: the Zaparax decoder (distance-biased windowed attention, state-space recurrence, experts with identity outputs,
+# looped layers) beside the Kifetar decoder (mixers, closes) and the Vazepel decoder (experts) at equal width / layer runs / vocabulary
+# ------------------------------------------------------------------------------------------------
+ZAPARAX_KERNELS = ("ssd_conv", "ssd_step", "pair_embed", "moe_glu") + KIFETAR_KERNELS
+
+
+def zaparax_config(width, vocab=32768, window=512):
+    """A realistic stack of 8 layer runs: state-space and attention layers in turn, six of them, the middle two looped twice; 2 x width
+    state-space columns in 64-wide heads with 128 x 64 states (8 heads per group), 128-wide attention heads (4 query heads per key / value
+    head), 28 gated experts of width / 4 and 4 identity experts (4 chosen) plus a shared expert of width / 2."""
+    H, Hs = width // 128, 2 * width // 64
+    sm = {"type": "mamba2", "mixer": {"heads": Hs, "vdim": 64, "state": 128, "groups": max(Hs // 8, 1), "conv": 4, "norm_groups": max(Hs // 8, 1)}}
+    at = {"type": "attention", "mixer": {"heads": H, "kv_heads": max(H // 4, 1), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+                                         "mask": {"size": window}, "q_temp": {"coef": 0.1, "every": 512}}}
+    moe = {"kind": "moe", "expert": {"ff": width // 4}, "router": {"experts": 28, "identity": 4, "top": 4}, "shared": {"ff": width // 2}}
+    return {"architecture": "Zaparax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5,
+            "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}}, "loop": {"start": 2, "stop": 4, "times": 2},
+            "layers": [{**(sm if i % 2 == 0 else at), "mlp": moe} for i in range(6)]}
+
+
+def _expert_rows_roofline(pk, runs, tokens, width, top, chosen, rf):
+    """The experts' row kernels of a prompt against the copy bandwidth: rows gathered (bf16 in and out), fp32 parts of the chosen experts
+    (`chosen` per token on average) and the shared expert's rows summed into fp32 rows."""
+    return {
+        "moe_gather": _roof(pk, ("moe_gather",), byts=runs * tokens * top * width * 4, **rf),
+        "moe_combine": _roof(pk, ("moe_combine",), byts=runs * tokens * width * 4 * (chosen + 2), **rf),
+        "moe_route": _roof(pk, ("moe_route",), byts=runs * tokens * (32 + 2 * top) * 4, **rf),
+        "moe_sort": _roof(pk, ("moe_sort",), byts=runs * tokens * top * 12, **rf),
+    }
+
+
+def measure_zaparax(dev, width, batch_prefill=4, prompt=2048, batch_decode=32, decode_steps=64, steps=5, warmup=3):
+    from vyomai_b200 import KifetarConfig, KifetarForCausalLM, VazepelConfig, VazepelForCausalLM, ZaparaxConfig, ZaparaxForCausalLM
+    hbm, _, _, src = peaks()
+    sms = torch.cuda.get_device_properties(dev).multi_processor_count
+    fp32_tflops = sms * 128 * 2 * 1.965e9 / 1e12
+    rf = dict(fp32_tflops=fp32_tflops, hbm=hbm)
+    tokens = batch_prefill * prompt
+    cfgd = zaparax_config(width)
+    cfg = ZaparaxConfig(cfgd)
+    model = ZaparaxForCausalLM(cfg, ZaparaxForCausalLM.random_weights(cfg, seed=0), dtype=torch.bfloat16, device=dev)
+    runs = [cfgd["layers"][i]["type"] for i in model.runs]
+    out = {"width": width, "layer_runs": runs, "vocab": cfg.vocab, "peaks": src, "fp32_tflops_nominal": round(fp32_tflops, 1)}
+    z = _packed_numbers(dev, model, cfg.vocab, batch_prefill, prompt, batch_decode, decode_steps, steps, warmup, kernels=ZAPARAX_KERNELS)
+    sm, at, moe = cfgd["layers"][0]["mixer"], cfgd["layers"][1]["mixer"], cfgd["layers"][0]["mlp"]
+    n_s, n_a = runs.count("mamba2"), runs.count("attention")
+    n_all = n_s + n_a
+    W = at["mask"]["size"]
+    pk, dk = z["prefill_kernels"], z["decode_kernels_eager"]
+    inner, gn = sm["heads"] * sm["vdim"], sm["groups"] * sm["state"]
+    state, chan = sm["heads"] * sm["state"] * sm["vdim"], inner + 2 * gn
+    top = moe["router"]["top"]
+    chosen = top * moe["router"]["experts"] / (moe["router"]["experts"] + moe["router"]["identity"])
+    vis = sum(min(p + 1, W) for p in range(prompt)) / prompt
+    z["prefill_roofline"] = {
+        "window_attn_tiled": _roof(pk, ("window_attn_tiled",), flop=n_a * tokens * at["heads"] * vis * (at["dim"] + at["vdim"]) * 2, **rf),
+        # per token and head: carried state read and updated (dim x vdim each), half a chunk of 64 inside it; counted as the fixed-decay form is
+        "linear_attn_chunk (state-space recurrence)": _roof(pk, ("linear_attn_chunk",), flop=n_s * tokens * sm["heads"] *
+                                                            (2 * sm["state"] * sm["vdim"] + 32 * (sm["state"] + sm["vdim"])) * 2, **rf),
+        "ssd_conv": _roof(pk, ("ssd_conv",), byts=n_s * tokens * chan * 8, **rf),
+        # a close reads residual and result, writes residual and the next norm (bf16); behind experts it also reads some bf16 input rows
+        "sandwich_norm": _roof(pk, ("sandwich_norm",), byts=2 * n_all * tokens * width * 14, **rf),
+        "rope_heads": _roof(pk, ("rope_heads",), byts=n_a * tokens * ((at["heads"] + at["kv_heads"]) * 8 + at["kv_heads"] * 8) * at["dim"], **rf),
+        "rms_norm (state-space read-out; fp32 in, bf16 out)": _roof(pk, ("rms_norm",), byts=n_s * tokens * inner * 6, **rf),
+        "pair_embed": _roof(pk, ("pair_embed",), byts=tokens * width * 8, **rf),
+        **_expert_rows_roofline(pk, n_all, tokens, width, top, chosen, rf),
+    }
+    z["decode_roofline"] = {
+        "window_attn_decode": _roof(dk, ("window_attn_decode", "window_attn_heads", "window_attn_heads_merge"),
+                                    byts=n_a * batch_decode * W * at["kv_heads"] * (at["dim"] + at["vdim"]) * 4, **rf),
+        "ssd_step (convolutions .. gated, normed read-out)": _roof(dk, ("ssd_step",), byts=n_s * batch_decode * (state * 8 + chan * (sm["conv"] + 1) * 4), **rf),
+        "sandwich_norm": _roof(dk, ("sandwich_norm",), byts=2 * n_all * batch_decode * width * 14, **rf),
+        "moe_glu": _roof(dk, ("moe_glu",), byts=n_all * batch_decode * ((moe["router"]["experts"] * moe["expert"]["ff"] + moe["shared"]["ff"]) * 2 +
+                                                                      (chosen * moe["expert"]["ff"] + moe["shared"]["ff"]) * 8), **rf),
+    }
+    per_run = {i: [L.inp.weight, L.mixer.o.weight, L.mlp.up_all.weight, L.mlp.down_all.weight, L.mlp.router_weight] for i, L in enumerate(model.layers)}
+    w_bytes = 2.0 * (sum(t.numel() for i in model.runs for t in per_run[i]) + model.head.weight.numel())
+    step_bytes = w_bytes + n_a * batch_decode * W * at["kv_heads"] * (at["dim"] + at["vdim"]) * 4 + n_s * batch_decode * state * 8
+    if z["decode"]["us_per_step_device"]:
+        z["decode"].update(step_algorithmic_MB=round(step_bytes / 1e6, 1),
+                           hbm_frac_device=round(step_bytes / (z["decode"]["us_per_step_device"] * 1e-6) / 1e9 / hbm, 3))
+    out["zaparax"] = z
+    del model
+    torch.cuda.empty_cache()
+    # the closest existing models. Mixers and closes: Kifetar (delta rule with one decay per head and windowed attention in turn, the same
+    # loop, dense feed-forward)
+    kd = kifetar_config(width)
+    kcfg = KifetarConfig(kd)
+    kmodel = KifetarForCausalLM(kcfg, KifetarForCausalLM.random_weights(kcfg, seed=0), dtype=torch.bfloat16, device=dev)
+    kz = _packed_numbers(dev, kmodel, kcfg.vocab, batch_prefill, prompt, batch_decode, decode_steps, steps, warmup, kernels=ZAPARAX_KERNELS)
+    dl, ka = kd["layers"][0]["mixer"], kd["layers"][1]["mixer"]
+    kpk, kdk = kz["prefill_kernels"], kz["decode_kernels_eager"]
+    kstate, kchan = dl["heads"] * dl["dim"] * dl["vdim"], 2 * dl["kv_heads"] * dl["dim"] + dl["heads"] * dl["vdim"]
+    kz["prefill_roofline"] = {
+        "window_attn_tiled": _roof(kpk, ("window_attn_tiled",), flop=n_a * tokens * ka["heads"] * vis * (ka["dim"] + ka["vdim"]) * 2, **rf),
+        "gd_scan (gated delta rule)": _roof(kpk, ("gd_scan",), flop=n_s * tokens * kstate * 7, **rf),
+        "gd_prep": _roof(kpk, ("gd_prep",), byts=n_s * tokens * (2 * kchan + 18 * dl["heads"]) * 4, **rf),
+        "sandwich_norm": _roof(kpk, ("sandwich_norm",), byts=2 * n_all * tokens * width * 14, **rf),
+        "rope_heads": _roof(kpk, ("rope_heads",), byts=n_a * tokens * ((ka["heads"] + ka["kv_heads"]) * 8 + ka["kv_heads"] * 8) * ka["dim"], **rf),
+        "rms_norm (delta read-out, gate)": _roof(kpk, ("rms_norm",), byts=n_s * tokens * dl["heads"] * dl["vdim"] * 10, **rf),
+        "embed_rows": _roof(kpk, ("embed_rows",), byts=tokens * width * 6, **rf),
+    }
+    kz["decode_roofline"] = {
+        "window_attn_decode": _roof(kdk, ("window_attn_decode", "window_attn_heads", "window_attn_heads_merge"),
+                                    byts=n_a * batch_decode * W * ka["kv_heads"] * (ka["dim"] + ka["vdim"]) * 4, **rf),
+        "gd_step": _roof(kdk, ("gd_step",), byts=n_s * batch_decode * (kstate * 8 + kchan * (dl["conv"] + 1) * 4), **rf),
+        "sandwich_norm": _roof(kdk, ("sandwich_norm",), byts=2 * n_all * batch_decode * width * 14, **rf),
+    }
+    out["kifetar"] = kz
+    del kmodel
+    torch.cuda.empty_cache()
+    # experts: Vazepel (softmax routing with groups, gated experts of the same sizes, 32 with weights)
+    vd = talking_config(width)
+    vcfg = VazepelConfig(vd)
+    vmodel = VazepelForCausalLM(vcfg, VazepelForCausalLM.random_weights(vcfg, seed=0), dtype=torch.bfloat16, device=dev)
+    vz = _packed_numbers(dev, vmodel, vcfg.vocab, batch_prefill, prompt, batch_decode, decode_steps, steps, warmup, kernels=ZAPARAX_KERNELS)
+    vm = vd["layers"][1]["mlp"]
+    v_moe = len(vd["layers"]) - 1
+    vtop = vm["router"]["top"]
+    vz["prefill_roofline"] = _expert_rows_roofline(vz["prefill_kernels"], v_moe, tokens, width, vtop, vtop, rf)
+    vz["decode_roofline"] = {"moe_glu": _roof(vz["decode_kernels_eager"], ("moe_glu",), byts=v_moe * batch_decode * (
+        (vm["router"]["experts"] * vm["expert"]["ff"] + vm["shared"]["ff"]) * 2 + (vtop * vm["expert"]["ff"] + vm["shared"]["ff"]) * 8), **rf)}
+    out["vazepel"] = vz
+    del vmodel
+    torch.cuda.empty_cache()
+    return out
+
+
+def run_zaparax(args):
+    from vyomai_b200 import _lib
+    if int(os.environ.get("WORLD_SIZE", "1")) > 1 or args.gpus != 1:
+        print(json.dumps({"workload": "zaparax", "error": "the Zaparax decoder measurement runs on one GPU"}))
+        return
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    L = _lib.lib()
+    sampler = ClockSampler(0)
+    sampler.start()
+    n0 = L.vy_launch_count()
+    res = [_guarded(measure_zaparax, dev, int(w), steps=max(args.steps // 2, 3), warmup=max(args.warmup, 3)) for w in args.hybrid_sizes.split(",")]
+    launches = L.vy_launch_count() - n0
+    sampler.stop_flag = True
+    sampler.join(timeout=2)
+    print(json.dumps({"workload": "zaparax", "metric": "zaparax_prefill_and_decode_tokens_per_s", "n_gpus": 1, "dtype": "bf16 (fp32 residual / scores / state)",
+                      "data": "synthetic", "sizes": res, "gpu_launches_total": int(launches), "gemm_poisoned": int(L.vy_gemm_poisoned()),
+                      "clocks": sampler.result(), "l2": "160 MB buffer rewritten between timed prefill iterations"}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1661,7 +1810,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--workload", default="package", choices=["package", "slots", "hybrid", "latent", "talking", "fubinex", "kifetar"],
+    ap.add_argument("--workload", default="package", choices=["package", "slots", "hybrid", "latent", "talking", "fubinex", "kifetar", "zaparax"],
                     help="package: VisionLanguageModel of the reference package (1 image token + 127 text, the headline); "
                          "slots: the notebook-II form (197 image tokens in a 248-token sequence); "
                          "hybrid: prefill / decode throughput of the Gelutar hybrid decoder beside DecoderModel at equal size (1 GPU, "
@@ -1669,8 +1818,9 @@ def main():
                          "latent: the same for the Zugunex latent-attention / mixture-of-experts decoder beside Gelutar at equal size; "
                          "talking: the same for the Vazepel parallel-layer decoder (score-exchanging attention heads) beside Zugunex; "
                          "fubinex: the same for the Fubinex decoder (latent / block-local / gated-linear / retention mixers) beside Gelutar; "
-                         "kifetar: the same for the Kifetar decoder (sigmoid-weighted attention / per-head-decay delta rule, looped layers) beside Gelutar")
-    ap.add_argument("--hybrid-sizes", default="1024,2048", help="--workload hybrid / latent / talking / fubinex / kifetar: model widths to measure")
+                         "kifetar: the same for the Kifetar decoder (sigmoid-weighted attention / per-head-decay delta rule, looped layers) beside Gelutar; "
+                         "zaparax: the same for the Zaparax decoder (distance-biased attention / state-space recurrence, experts) beside Kifetar and Vazepel")
+    ap.add_argument("--hybrid-sizes", default="1024,2048", help="--workload hybrid / latent / talking / fubinex / kifetar / zaparax: model widths to measure")
     ap.add_argument("--no-configs-1-2", action="store_true", help="skip the encoder (C1) / ViT (C2) measurements appended at N = 1")
     ap.add_argument("--no-config5", action="store_true", help="skip the PaliGemma-scale prefill + decode measurement appended at N = 1")
     ap.add_argument("--no-slots", action="store_true", help="skip the notebook-II measurement appended at N = 1")
@@ -1695,6 +1845,8 @@ def main():
         run_fubinex(args)
     elif args.workload == "kifetar":
         run_kifetar(args)
+    elif args.workload == "zaparax":
+        run_zaparax(args)
     else:
         run_ours(args)
 

@@ -18,6 +18,7 @@ Differences from the notebook, on purpose:
 """
 from __future__ import annotations
 
+import gc
 import itertools
 from collections import deque
 
@@ -338,10 +339,15 @@ class _CapturedStep:
         self.graph = torch.cuda.CUDAGraph()
         pdl = os.environ.get("VY_DECODE_PDL", "1") != "0"   # each short kernel's launch overlaps its predecessor's tail
         prev = _lib.lib().vy_set_pdl(1) if pdl else None
+        # a garbage collection inside the capture could free an older engine's graph or pools, which invalidates the capture
+        collecting = gc.isenabled()
+        gc.disable()
         try:
             with torch.cuda.graph(self.graph), torch.no_grad():
                 self.logits = engine.model.step(ids_t, batch, engine.cache.views, rows_t)
         finally:
+            if collecting:
+                gc.enable()
             if pdl:
                 _lib.lib().vy_set_pdl(prev)
 
