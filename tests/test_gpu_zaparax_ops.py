@@ -336,13 +336,21 @@ def _ssd_op(cuts, *, H=4, G=2, N=9, dv=10, taps=3, ng=2, seed=20, dt_shift=0.0, 
 
 @pytest.mark.parametrize("kw", [dict(), dict(H=3, G=1, N=40, dv=33, taps=4, ng=3), dict(H=2, G=2, N=130, dv=8, taps=7, ng=1), dict(H=6, G=2, N=16, dv=140, taps=2, ng=4),
                                 dict(H=1, G=1, N=1, dv=2, taps=1, ng=1), dict(H=20, G=4, N=64, dv=12, taps=16, ng=20), dict(H=4, G=1, N=128, dv=64, taps=4, ng=1, wdt=torch.bfloat16),
-                                dict(H=2, G=1, N=8, dv=600, taps=3, ng=5), dict(H=1, G=1, N=3, dv=301, taps=2, ng=7), dict(bias=False, gate=False)])
+                                dict(H=8, G=2, N=128, dv=64, taps=4, ng=2), dict(H=4, G=2, N=64, dv=128, taps=3, ng=2), dict(H=2, G=2, N=256, dv=16, taps=4, ng=1), dict(H=2, G=1, N=8, dv=600, taps=3, ng=5), dict(H=1, G=1, N=3, dv=301, taps=2, ng=7), dict(bias=False, gate=False)])
 def test_state_space_over_a_packed_batch(kw):
     """Unequal sequences side by side: prompts over several chunks, portions that end off the chunks, a sequence of one token, single tokens
     beside portions, then single tokens only (their own kernel); states, groups, norm groups and taps of unrelated sizes."""
     cuts = [[141, 1, 1], [6, 64, 1, 1], [1, 1, 1], [3, 2, 70, 1, 1, 1]]
     for got, want, st, ost in _ssd_op(cuts, **kw):
         assert HU.rel_err(got, want) < 1e-4 and HU.rel_err(st, ost) < 2e-5
+
+
+@pytest.mark.parametrize("H,G,N,dv", [(4, 2, 9, 10), (8, 1, 16, 8), (8, 1, 5, 3), (12, 3, 20, 32), (8, 2, 64, 64), (4, 1, 32, 128), (6, 3, 256, 32)])
+def test_state_space_single_tokens_of_many_sequences(H, G, N, dv):
+    """Batches large enough that a CTA takes two or four heads of a group."""
+    cuts = [[1 + s % 3, 1, 1] for s in range(230)]
+    got, want, st, ost = (torch.cat(x) if x[0].dim() == 2 else torch.stack(x) for x in zip(*_ssd_op(cuts, H=H, G=G, N=N, dv=dv)))
+    assert HU.rel_err(got, want) < 1e-4 and HU.rel_err(st, ost) < 2e-5
 
 
 @pytest.mark.parametrize("cuts", [[100], [37, 63], [1] * 40])
