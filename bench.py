@@ -1706,7 +1706,7 @@ def measure_zaparax(dev, width, batch_prefill=4, prompt=2048, batch_decode=32, d
     pk, dk = z["prefill_kernels"], z["decode_kernels_eager"]
     inner, gn = sm["heads"] * sm["vdim"], sm["groups"] * sm["state"]
     state, chan = sm["heads"] * sm["state"] * sm["vdim"], inner + 2 * gn
-    top = moe["router"]["top"]
+    top, ff_e = moe["router"]["top"], moe["expert"]["ff"]
     chosen = top * moe["router"]["experts"] / (moe["router"]["experts"] + moe["router"]["identity"])
     vis = sum(min(p + 1, W) for p in range(prompt)) / prompt
     z["prefill_roofline"] = {
@@ -1720,6 +1720,8 @@ def measure_zaparax(dev, width, batch_prefill=4, prompt=2048, batch_decode=32, d
         "rope_heads": _roof(pk, ("rope_heads",), byts=n_a * tokens * ((at["heads"] + at["kv_heads"]) * 8 + at["kv_heads"] * 8) * at["dim"], **rf),
         "rms_norm (state-space read-out; fp32 in, bf16 out)": _roof(pk, ("rms_norm",), byts=n_s * tokens * inner * 6, **rf),
         "pair_embed": _roof(pk, ("pair_embed",), byts=tokens * width * 8, **rf),
+        # all experts over all rows: unchosen columns are written 0 unread, chosen ones and the shared expert's read and written (bf16)
+        "moe_scale": _roof(pk, ("moe_scale",), byts=n_all * tokens * (moe["router"]["experts"] * ff_e + chosen * ff_e + 2 * moe["shared"]["ff"]) * 2, **rf),
         **_expert_rows_roofline(pk, n_all, tokens, width, top, chosen, rf),
     }
     z["decode_roofline"] = {
@@ -1775,6 +1777,9 @@ def measure_zaparax(dev, width, batch_prefill=4, prompt=2048, batch_decode=32, d
     v_moe = len(vd["layers"]) - 1
     vtop = vm["router"]["top"]
     vz["prefill_roofline"] = _expert_rows_roofline(vz["prefill_kernels"], v_moe, tokens, width, vtop, vtop, rf)
+    if "moe_sort" not in vz["prefill_kernels"]:   # all experts over all rows: fp32 pre-activations of the chosen in, all columns out (bf16)
+        vz["prefill_roofline"]["moe_glu"] = _roof(vz["prefill_kernels"], ("moe_glu",), byts=v_moe * tokens * (
+            (vm["router"]["experts"] * vm["expert"]["ff"] + vm["shared"]["ff"]) * 2 + (vtop * vm["expert"]["ff"] + vm["shared"]["ff"]) * 8), **rf)
     vz["decode_roofline"] = {"moe_glu": _roof(vz["decode_kernels_eager"], ("moe_glu",), byts=v_moe * batch_decode * (
         (vm["router"]["experts"] * vm["expert"]["ff"] + vm["shared"]["ff"]) * 2 + (vtop * vm["expert"]["ff"] + vm["shared"]["ff"]) * 8), **rf)}
     out["vazepel"] = vz

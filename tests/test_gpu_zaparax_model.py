@@ -26,11 +26,15 @@ FP32_TOL = 2e-4
 
 
 class Ref:
-    """The oracle's logits of one token sequence and, for bfloat16 models, the limit that rounding sets."""
+    """The oracle's logits of one token sequence and, for bfloat16 models, the limit that rounding sets. `drawn`: a configuration nobody
+    chose, which may amplify roundings (a norm over a few columns that cancel): its float32 limit grows with what rounding every product's
+    input to float32, one of many roundings, does in the oracle."""
 
-    def __init__(self, cfg, W, toks, dtype, fp32_tol=FP32_TOL):
+    def __init__(self, cfg, W, toks, dtype, fp32_tol=FP32_TOL, drawn=False):
         self.logits = O.forward(cfg, W, toks)
         self.tol = fp32_tol
+        if drawn and dtype == torch.float32:
+            self.tol = max(fp32_tol, 60.0 * HU.rel_err(O.forward(cfg, W, toks, rnd=lambda x: x.float().double()), self.logits))
         if dtype == torch.bfloat16:
             self.tol = max(2e-2, 3.0 * HU.rel_err(O.forward(cfg, W, toks, rnd=O.to_bf16), self.logits))
 
@@ -236,6 +240,17 @@ def test_experts_sorted_by_row(dtype, cfg_name):
     _check(HU.feed_in_portions(eng, "s", toks, [19, 2, 14]), Ref(cfg, W, toks, dtype))
 
 
+@pytest.mark.parametrize("kind", ["attention", "mamba2"])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_models_of_one_mixer_and_an_odd_width(kind, dtype):
+    """Only pages or only state slots to manage; rows that no 16-byte access fits."""
+    cfg = U.config([U.layer(kind, U.attention() if kind == "attention" else U.mamba(), f) for f in (U.moe(), None)], width=37, vocab=61, loop=(0, 1, 2))
+    model, W = U.build(cfg, dtype=dtype)
+    eng, _ = HU.engine_for(model)
+    toks = HU.tokens(40, cfg["vocab"], 52)
+    _check(HU.feed_in_portions(eng, "s", toks, [17, 2, 9]), Ref(cfg, W, toks, dtype))
+
+
 @pytest.mark.parametrize("loop", [None, (0, 2, 1), (0, 2, 2), (1, 2, 3), (0, 1, 2)])
 def test_loops(loop):
     """No loop, a loop over all layers (one pass is no loop), over the last, over the first; a pass reads its own cache, so the passes of a
@@ -253,7 +268,7 @@ def test_loops(loop):
         assert HU.rel_err(O.forward({**cfg, "loop": None}, W, toks), ref) > 1e-2
 
 
-@pytest.mark.parametrize("seed", range(10))
+@pytest.mark.parametrize("seed", range(16))
 def test_configurations_drawn_at_random(seed):
     """Other layer orders, loops, head counts, channel counts, windows, constants: a prompt with decoding, portions, and two unequal
     requests in one batch, in fp32 and in bf16 (tensor-core products wherever the drawn sizes allow them) against the oracle."""
@@ -261,7 +276,7 @@ def test_configurations_drawn_at_random(seed):
         cfg = U.random_config(seed)
         toks, other = HU.tokens(70, cfg["vocab"], 40 + seed), HU.tokens(21, cfg["vocab"], 80 + seed)
         model, W = U.build(cfg, dtype=dtype, seed=seed)
-        ref, ref_o = Ref(cfg, W, toks, dtype, fp32_tol=4e-4), Ref(cfg, W, other, dtype, fp32_tol=4e-4)
+        ref, ref_o = Ref(cfg, W, toks, dtype, drawn=True), Ref(cfg, W, other, dtype, drawn=True)
         eng, _ = HU.engine_for(model, block_size=16)
         _check(HU.feed_in_portions(eng, "w", toks, [40]), ref, "prompt + decoding")
         _check(HU.feed_in_portions(eng, "p", toks, [19, 2, 30, 7]), ref, "portions")

@@ -122,5 +122,5 @@ def random_config(seed: int) -> dict:
         a = int(torch.randint(0, n, (1,), generator=g))
         b = int(torch.randint(a + 1, n + 1, (1,), generator=g))
         loop = (a, b, pick([1, 2, 3]))
-    return config(layers, width=pick([48, 64, 96, 160]), vocab=pick([50, 131, 256]), eps=pick([1e-6, 1e-5]), loop=loop,
+    return config(layers, width=pick([37, 48, 64, 100, 160]), vocab=pick([50, 131, 256]), eps=pick([1e-6, 1e-5]), loop=loop,
                   bigram=pick([None, (1, 5, 9), (17, 31, 2), (211, 10 ** 12 + 39, 2 ** 40 + 1)]), scale=pick([1.0, 3.0, 0.5]))
